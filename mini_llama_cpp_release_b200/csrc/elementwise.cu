@@ -320,46 +320,151 @@ __global__ void convert_kernel(const TIn* __restrict__ in, long long total, TOut
     if (idx < total) out[idx] = from_float<TOut>(to_float(in[idx]));
 }
 
-// ------------------------------------------------------------------ layer norm (gain, no bias)
-// LN(v) = (v - mean(v)) / sqrt(mean((v - mean)²) + eps) · w, statistics in float32 in two passes (the mean first,
-// then the squared deviations).  A block per row; the row waits in shared memory between the passes.
+// ------------------------------------------------------------------ layer norm (gain, optional bias)
+// LN(v) = (v - mean(v)) / sqrt(mean((v - mean)²) + eps) · w + b, statistics in float32 in two passes (the mean first,
+// then the squared deviations).  b may be null (no bias).
 //
-// ln_mode 0, "norm of the stream":   x += sum of the delta slices (if any);  out = LN(x)            (out in T)
-// ln_mode 1, "norm of the branch":   x += LN(sum of the y slices);           out = x, if asked for  (out in T)
+// ln_mode 0, "norm of the stream":   x += branch (if any);  out = LN(x)            (out in T)
+// ln_mode 1, "norm of the branch":   x += LN(branch);       out = x, if asked for  (out in T)
+//
+// The branch is y, float32 slices added in order, or the weighted sum of a token's expert rows,
+// sum_j weights[t][j] · rows[row_of[t][j]], j in the order of the choices.
+struct NormBranch {
+    const float* y;             // [n_slices][n][d], or null
+    int n_slices;
+    long long slice_stride;
+    const float* rows;          // expert rows [.][d], or null
+    const int* row_of;          // [n][top]
+    const float* weights;       // [n][top]
+    int top;
+};
+
+struct Four { float e[4]; };
+__device__ __forceinline__ Four load_four(const float* p) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    return Four{{t.x, t.y, t.z, t.w}};
+}
+
+// v (VEC entries of row t from entry i on) += the branch's entries
+template <int VEC>
+__device__ __forceinline__ void add_branch(const NormBranch& br, long long t, int d, int i, float (&v)[VEC]) {
+    if (br.y != nullptr) {
+        const float* p = br.y + t * d + i;
+#pragma unroll 8
+        for (int s = 0; s < br.n_slices; ++s) {
+            if constexpr (VEC == 4) {
+                const Four q = load_four(p + s * br.slice_stride);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) v[k] += q.e[k];
+            } else {
+                v[0] += __ldg(p + s * br.slice_stride);
+            }
+        }
+    }
+    if (br.rows != nullptr) {
+        float acc[VEC];
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) acc[k] = 0.0f;
+#pragma unroll 4
+        for (int j = 0; j < br.top; ++j) {
+            const float w = br.weights[t * br.top + j];
+            const float* p = br.rows + (long long)br.row_of[t * br.top + j] * d + i;
+            if constexpr (VEC == 4) {
+                const Four q = load_four(p);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w, q.e[k], acc[k]);
+            } else {
+                acc[0] = fmaf(w, *p, acc[0]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) v[k] += acc[k];
+    }
+}
+
 template <typename T>
-__global__ void layernorm_kernel(float* __restrict__ x, const float* __restrict__ y, int n_slices, long long slice_stride,
-                                 const float* __restrict__ gain, float eps, int d, int ln_mode, T* __restrict__ out) {
-    extern __shared__ float row[];
+__device__ __forceinline__ void store_four(T* p, const float (&r)[4]) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]);
+    } else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+    }
+}
+
+// A block per row; the row waits in shared memory between the passes.  VEC 4: 16-byte accesses (rows whose length is a
+// multiple of 4, all pointers 16-byte aligned); VEC 1: any row, and few rows, where one entry a thread has more loads in flight.
+template <typename T, int VEC>
+__global__ void layernorm_kernel(float* __restrict__ x, NormBranch br, const float* __restrict__ gain,
+                                 const float* __restrict__ bias, float eps, int d, int ln_mode, T* __restrict__ out) {
+    extern __shared__ __align__(16) float row[];
     __shared__ float scratch[32];
     grid_launch_dependents();
     grid_dependency_wait();
-    const long long base = (long long)blockIdx.x * d;
+    const long long t = blockIdx.x, base = t * d;
+    const bool has_branch = br.y != nullptr || br.rows != nullptr;
     float sum = 0.0f;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        float v = (ln_mode == 0) ? x[base + i] : 0.0f;
-        if (y != nullptr) {
-#pragma unroll 8
-            for (int s = 0; s < n_slices; ++s) v += __ldg(y + s * slice_stride + base + i);
+    for (int i = threadIdx.x * VEC; i < d; i += blockDim.x * VEC) {
+        float v[VEC];
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) v[k] = 0.0f;
+        if (ln_mode == 0) {
+            if constexpr (VEC == 4) {
+                const Four q = load_four(x + base + i);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) v[k] = q.e[k];
+            } else {
+                v[0] = x[base + i];
+            }
         }
-        if (ln_mode == 0 && y != nullptr) x[base + i] = v;
-        row[i] = v;
-        sum += v;
+        if (has_branch) {
+            add_branch<VEC>(br, t, d, i, v);
+            if (ln_mode == 0) {
+                if constexpr (VEC == 4) store_four<float>(x + base + i, v);
+                else x[base + i] = v[0];
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            row[i + k] = v[k];
+            sum += v[k];
+        }
     }
     const float mean = block_sum(sum, scratch) / (float)d;
     float sq = 0.0f;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        const float c = row[i] - mean;
-        sq += c * c;
-    }
+    for (int i = threadIdx.x * VEC; i < d; i += blockDim.x * VEC)
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            const float c = row[i + k] - mean;
+            sq += c * c;
+        }
     const float rstd = 1.0f / sqrtf(block_sum(sq, scratch) / (float)d + eps);
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        const float v = (row[i] - mean) * rstd * gain[i];
-        if (ln_mode == 0) {
-            out[base + i] = from_float<T>(v);
+    for (int i = threadIdx.x * VEC; i < d; i += blockDim.x * VEC) {
+        float r[VEC];
+        if constexpr (VEC == 4) {
+            const Four g = load_four(gain + i);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) r[k] = (row[i + k] - mean) * rstd * g.e[k];
+            if (bias != nullptr) {
+                const Four b = load_four(bias + i);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) r[k] += b.e[k];
+            }
+            if (ln_mode != 0) {
+                const Four xo = load_four(x + base + i);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) r[k] = xo.e[k] + r[k];
+                store_four<float>(x + base + i, r);
+            }
+            if (out != nullptr) store_four<T>(out + base + i, r);
         } else {
-            const float nx = x[base + i] + v;
-            x[base + i] = nx;
-            if (out != nullptr) out[base + i] = from_float<T>(nx);
+            r[0] = (row[i] - mean) * rstd * gain[i];
+            if (bias != nullptr) r[0] += bias[i];
+            if (ln_mode != 0) {
+                r[0] = x[base + i] + r[0];
+                x[base + i] = r[0];
+            }
+            if (out != nullptr) out[base + i] = from_float<T>(r[0]);
         }
     }
 }
@@ -368,8 +473,8 @@ __global__ void layernorm_kernel(float* __restrict__ x, const float* __restrict_
 // d <= 128 * NV, d a multiple of 4, all pointers 16-byte aligned); no shared memory and no block-wide barrier.
 template <typename T, int NV>
 __global__ void __launch_bounds__(256)
-layernorm_warp_kernel(float* __restrict__ x, const float* __restrict__ y, int n_slices, long long slice_stride,
-                      const float* __restrict__ gain, float eps, int d, int n, int ln_mode, T* __restrict__ out) {
+layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restrict__ gain, const float* __restrict__ bias,
+                      float eps, int d, int n, int ln_mode, T* __restrict__ out) {
     grid_launch_dependents();
     grid_dependency_wait();
     const int lane = threadIdx.x & 31;
@@ -377,6 +482,7 @@ layernorm_warp_kernel(float* __restrict__ x, const float* __restrict__ y, int n_
     if (row >= n) return;
     const long long base = (long long)row * d;
     const int d4 = d >> 2;
+    const bool has_branch = br.y != nullptr || br.rows != nullptr;
     float4* x4 = reinterpret_cast<float4*>(x + base);
     float4 v[NV], xv[NV];
 #pragma unroll
@@ -385,9 +491,9 @@ layernorm_warp_kernel(float* __restrict__ x, const float* __restrict__ y, int n_
         xv[k] = (i < d4) ? x4[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         v[k] = (ln_mode == 0) ? xv[k] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     }
-    if (y != nullptr) {
-        for (int s = 0; s < n_slices; ++s) {
-            const float4* t4 = reinterpret_cast<const float4*>(y + s * slice_stride + base);
+    if (br.y != nullptr) {
+        for (int s = 0; s < br.n_slices; ++s) {
+            const float4* t4 = reinterpret_cast<const float4*>(br.y + s * br.slice_stride + base);
 #pragma unroll
             for (int k = 0; k < NV; ++k) {
                 const int i = lane + 32 * k;
@@ -397,6 +503,26 @@ layernorm_warp_kernel(float* __restrict__ x, const float* __restrict__ y, int n_
                 }
             }
         }
+    }
+    if (br.rows != nullptr) {
+        float4 acc[NV];
+#pragma unroll
+        for (int k = 0; k < NV; ++k) acc[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int j = 0; j < br.top; ++j) {
+            const float w = br.weights[(long long)row * br.top + j];
+            const float4* t4 = reinterpret_cast<const float4*>(br.rows + (long long)br.row_of[(long long)row * br.top + j] * d);
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                const int i = lane + 32 * k;
+                if (i < d4) {
+                    const float4 t = __ldg(t4 + i);
+                    acc[k].x = fmaf(w, t.x, acc[k].x); acc[k].y = fmaf(w, t.y, acc[k].y);
+                    acc[k].z = fmaf(w, t.z, acc[k].z); acc[k].w = fmaf(w, t.w, acc[k].w);
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < NV; ++k) { v[k].x += acc[k].x; v[k].y += acc[k].y; v[k].z += acc[k].z; v[k].w += acc[k].w; }
     }
     float sum = 0.0f;
 #pragma unroll
@@ -412,38 +538,49 @@ layernorm_warp_kernel(float* __restrict__ x, const float* __restrict__ y, int n_
     }
     const float rstd = 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
     const float4* g4 = reinterpret_cast<const float4*>(gain);
+    const float4* b4 = reinterpret_cast<const float4*>(bias);
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = lane + 32 * k;
         if (i >= d4) continue;
         const float4 g = __ldg(g4 + i);
-        float4 r = make_float4((v[k].x - mean) * rstd * g.x, (v[k].y - mean) * rstd * g.y, (v[k].z - mean) * rstd * g.z,
-                               (v[k].w - mean) * rstd * g.w);
+        float r[4] = {(v[k].x - mean) * rstd * g.x, (v[k].y - mean) * rstd * g.y, (v[k].z - mean) * rstd * g.z,
+                      (v[k].w - mean) * rstd * g.w};
+        if (b4 != nullptr) {
+            const float4 b = __ldg(b4 + i);
+            r[0] += b.x; r[1] += b.y; r[2] += b.z; r[3] += b.w;
+        }
         if (ln_mode == 0) {
-            if (y != nullptr) x4[i] = v[k];
+            if (has_branch) x4[i] = v[k];
         } else {
-            r = make_float4(xv[k].x + r.x, xv[k].y + r.y, xv[k].z + r.z, xv[k].w + r.w);
-            x4[i] = r;
+            r[0] += xv[k].x; r[1] += xv[k].y; r[2] += xv[k].z; r[3] += xv[k].w;
+            x4[i] = make_float4(r[0], r[1], r[2], r[3]);
             if (out == nullptr) continue;
         }
-        if (sizeof(T) == 4) {
-            reinterpret_cast<float4*>(out + base)[i] = r;
-        } else {
-            __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
-            reinterpret_cast<uint2*>(out + base)[i] = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
-        }
+        store_four<T>(out + base + 4 * i, r);
     }
 }
 
 template <typename T>
-static cudaError_t launch_layernorm_warp(int nv, float* x, const float* y, int n_slices, long long stride, const float* gain,
-                                         float eps, int d, int n, int ln_mode, T* out, cudaStream_t s) {
-    const dim3 grid((n + 7) / 8), block(256);
-    if (nv <= 1) return launch_pdl(layernorm_warp_kernel<T, 1>, grid, block, 0, s, x, y, n_slices, stride, gain, eps, d, n, ln_mode, out);
-    if (nv <= 2) return launch_pdl(layernorm_warp_kernel<T, 2>, grid, block, 0, s, x, y, n_slices, stride, gain, eps, d, n, ln_mode, out);
-    if (nv <= 4) return launch_pdl(layernorm_warp_kernel<T, 4>, grid, block, 0, s, x, y, n_slices, stride, gain, eps, d, n, ln_mode, out);
-    if (nv <= 8) return launch_pdl(layernorm_warp_kernel<T, 8>, grid, block, 0, s, x, y, n_slices, stride, gain, eps, d, n, ln_mode, out);
-    return launch_pdl(layernorm_warp_kernel<T, 12>, grid, block, 0, s, x, y, n_slices, stride, gain, eps, d, n, ln_mode, out);
+static cudaError_t launch_layernorm(bool vec, int nv, float* x, const NormBranch& br, const float* gain, const float* bias, float eps,
+                                    int d, int n, int ln_mode, T* out, size_t smem, int threads, cudaStream_t s) {
+    if (vec && nv <= 12 && n >= 128) {
+        const dim3 grid((n + 7) / 8), block(256);
+        auto k = nv <= 1 ? layernorm_warp_kernel<T, 1> : nv <= 2 ? layernorm_warp_kernel<T, 2> : nv <= 4 ? layernorm_warp_kernel<T, 4>
+               : nv <= 8 ? layernorm_warp_kernel<T, 8> : layernorm_warp_kernel<T, 12>;
+        return launch_pdl(k, grid, block, 0, s, x, br, gain, bias, eps, d, n, ln_mode, out);
+    }
+    static bool raised = false;
+    if (smem > 48 * 1024 && !raised) {
+        for (auto k : {layernorm_kernel<T, 1>, layernorm_kernel<T, 4>}) {
+            cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
+            if (e != cudaSuccess) return e;
+        }
+        raised = true;
+    }
+    if (vec && n >= 128)
+        return launch_pdl(layernorm_kernel<T, 4>, dim3(n), dim3(threads), smem, s, x, br, gain, bias, eps, d, ln_mode, out);
+    return launch_pdl(layernorm_kernel<T, 1>, dim3(n), dim3(threads), smem, s, x, br, gain, bias, eps, d, ln_mode, out);
 }
 
 // ------------------------------------------------------------------ per-head RMS norm, partial rotation, cache write
@@ -457,13 +594,16 @@ static cudaError_t launch_layernorm_warp(int nv, float* x, const float* y, int n
 // Options of the kernel below beyond its first form: biases added to the projection's columns as they are read (null:
 // none); `whole_row`: the norm's statistic is taken over all query heads together (and over all key heads together) and the
 // gains are as long as the projection, instead of one statistic per head and a gain shared by the heads; `interleaved`: the
-// rotation pairs entry 2j with 2j + 1 instead of entry j with j + dims/2.
+// rotation pairs entry 2j with 2j + 1 instead of entry j with j + dims/2; `temp_every` > 0: the queries of position p are
+// multiplied by 1 + temp_coef · ln(floor((p + 1) / temp_every) + 1).
 struct QkOptions {
     const float* q_bias;
     const float* k_bias;
     const float* v_bias;
     int whole_row;
     int interleaved;
+    float temp_coef;
+    int temp_every;
 };
 
 template <typename T>
@@ -481,6 +621,7 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
     const int half = rot_dims >> 1;
     const float2* cs = (rope != nullptr && half > 0) ? rope + (long long)min(p, rope_positions - 1) * half : nullptr;
     const int n_heads = q_heads + 2 * kv_heads_in_row;
+    const float q_temp = opt.temp_every > 0 ? 1.0f + opt.temp_coef * logf((float)((p + 1) / opt.temp_every) + 1.0f) : 1.0f;
     // a norm over the whole projection: one statistic for all query heads and one for all key heads, summed in an order
     // that the row's length alone fixes (a thread a strided share, then the block's tree)
     __shared__ float scratch[32];
@@ -522,6 +663,7 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
                 ss = warp_sum(ss);
                 f = eps >= 0.0f ? 1.0f / sqrtf(ss / (float)dim + eps) : 1.0f;      // a negative eps: no norm
             }
+            if (is_q) f *= q_temp;              // the rotation is linear: the factor acts on both entries of a pair
             for (int i = lane; i < D; i += 32) {
                 float v = 0.0f;
                 if (i < dim) {
@@ -620,39 +762,30 @@ extern "C" int mlc_add_rmsnorm(float* x, const float* delta, int n_slices, const
     return 0;
 }
 
-// ln_mode 0: x += sum of the n_slices slices of y (if y is given), out = LN(x)·gain in out_dtype.
-// ln_mode 1: x += LN(sum of the slices of y)·gain; out (may be null) = the new x in out_dtype.
-extern "C" int mlc_layernorm(float* x, const float* y, int n_slices, const float* gain, float eps, int n, int d, int ln_mode,
-                             void* out, int out_dtype, void* stream) {
+// ln_mode 0: x += branch (if y or rows is given), out = LN(x)·gain + bias in out_dtype.
+// ln_mode 1: x += LN(branch)·gain + bias; out (may be null) = the new x in out_dtype.
+// The branch: y (n_slices slices of n·d floats), or rows / row_of / weights / top (a token's expert rows); bias may be null.
+extern "C" int mlc_layernorm(float* x, const float* y, int n_slices, const float* rows, const int* row_of, const float* weights,
+                             int top, const float* gain, const float* bias, float eps, int n, int d, int ln_mode, void* out,
+                             int out_dtype, void* stream) {
     if (n <= 0) return 0;
     if (d <= 0 || d > 32768 || (y != nullptr && n_slices < 1) || (ln_mode != 0 && ln_mode != 1)) return MLC_ERR_BAD_SIZE;
-    if ((ln_mode == 1 && y == nullptr) || (ln_mode == 0 && out == nullptr)) return MLC_ERR_BAD_SIZE;
+    if (rows != nullptr && (y != nullptr || row_of == nullptr || weights == nullptr || top < 1)) return MLC_ERR_BAD_SIZE;
+    if ((ln_mode == 1 && y == nullptr && rows == nullptr) || (ln_mode == 0 && out == nullptr)) return MLC_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
-    const long long stride = (long long)n * d;
+    const NormBranch br{y, n_slices, (long long)n * d, rows, row_of, weights, top};
     const size_t smem = (size_t)d * sizeof(float);
-    static bool raised = false;
-    if (smem > 48 * 1024 && !raised) {
-        cudaError_t e1 = cudaFuncSetAttribute(layernorm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
-        cudaError_t e2 = cudaFuncSetAttribute(layernorm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
-        if (e1 != cudaSuccess) return (int)e1;
-        if (e2 != cudaSuccess) return (int)e2;
-        raised = true;
-    }
-    cudaError_t e;
-    if (out_dtype != MLC_DTYPE_F32 && out_dtype != MLC_DTYPE_BF16) return MLC_ERR_BAD_DTYPE;
     const int nv = ((d >> 2) + 31) / 32;                 // 16-byte pieces per lane if a warp takes a row
-    const bool vec = (d & 3) == 0 && ((((uintptr_t)x) | ((uintptr_t)y) | ((uintptr_t)gain) | ((uintptr_t)out)) & 15) == 0;
-    if (vec && nv <= 12 && n >= 128) {
-        e = out_dtype == MLC_DTYPE_F32
-                ? launch_layernorm_warp<float>(nv, x, y, n_slices, stride, gain, eps, d, n, ln_mode, (float*)out, s)
-                : launch_layernorm_warp<bf16>(nv, x, y, n_slices, stride, gain, eps, d, n, ln_mode, (bf16*)out, s);
-        return e == cudaSuccess ? 0 : (int)e;
-    }
-    const int threads = norm_threads(d, n);
+    const bool vec = (d & 3) == 0 && ((((uintptr_t)x) | ((uintptr_t)y) | ((uintptr_t)rows) | ((uintptr_t)gain) | ((uintptr_t)bias) |
+                                       ((uintptr_t)out)) & 15) == 0;
+    const int threads = vec && n >= 128 ? norm_threads(d >> 2, n) : norm_threads(d, n);
+    cudaError_t e;
     if (out_dtype == MLC_DTYPE_F32)
-        e = launch_pdl(layernorm_kernel<float>, dim3(n), dim3(threads), smem, s, x, y, n_slices, stride, gain, eps, d, ln_mode, (float*)out);
+        e = launch_layernorm<float>(vec, nv, x, br, gain, bias, eps, d, n, ln_mode, (float*)out, smem, threads, s);
+    else if (out_dtype == MLC_DTYPE_BF16)
+        e = launch_layernorm<bf16>(vec, nv, x, br, gain, bias, eps, d, n, ln_mode, (bf16*)out, smem, threads, s);
     else
-        e = launch_pdl(layernorm_kernel<bf16>, dim3(n), dim3(threads), smem, s, x, y, n_slices, stride, gain, eps, d, ln_mode, (bf16*)out);
+        return MLC_ERR_BAD_DTYPE;
     return e == cudaSuccess ? 0 : (int)e;
 }
 
@@ -662,9 +795,10 @@ extern "C" int mlc_qk_norm_rope_cache(const float* proj, long long stride, int q
                                       int kv_heads_in_row, int dim, int vdim, int D, float v_scale, void* q_out, int dtype,
                                       void* k_pool, void* v_pool, const int* page_table, long long entry_offset,
                                       int pages_per_seq, int page_size, int cache_kv_heads, const float* q_bias,
-                                      const float* k_bias, const float* v_bias, int whole_row, int interleaved, void* stream) {
+                                      const float* k_bias, const float* v_bias, int whole_row, int interleaved, float temp_coef,
+                                      int temp_every, void* stream) {
     if (n <= 0) return 0;
-    const QkOptions opt{q_bias, k_bias, v_bias, whole_row, interleaved};
+    const QkOptions opt{q_bias, k_bias, v_bias, whole_row, interleaved, temp_coef, temp_every};
     if (dim <= 0 || vdim <= 0 || D < dim || D < vdim || q_heads <= 0 || kv_heads_in_row < 0) return MLC_ERR_BAD_SIZE;
     if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim) return MLC_ERR_BAD_SIZE;
     if (kv_heads_in_row != 0 && kv_heads_in_row != cache_kv_heads) return MLC_ERR_BAD_SIZE;

@@ -84,11 +84,12 @@ constexpr int HP_K = 16;
 
 // out[t][h][j] = sum_d in[t][h][d] · W[h][d][j] for j < n_out, d < n_in; every operand by strides (in elements):
 // in at t*in_st + h*in_sh + d, W at h*w_sh + d*w_sd + j*w_sj, out at t*out_st + h*out_sh + j.
+// `gate` (float32 rows of stride gate_st, or null): out is multiplied by sigmoid(gate[t][h*n_out + j]) before it is rounded.
 template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 head_project_kernel(const TI* __restrict__ in, long long in_st, long long in_sh, const TW* __restrict__ w, long long w_sh,
                     long long w_sd, long long w_sj, TO* __restrict__ out, long long out_st, long long out_sh, int n, int n_in,
-                    int n_out) {
+                    int n_out, const float* __restrict__ gate, long long gate_st) {
     const int h = blockIdx.z;
     const int t0 = blockIdx.y * HP_TILE, j0 = blockIdx.x * HP_TILE;
     __shared__ float xs[HP_K][HP_TILE + 1];
@@ -129,7 +130,10 @@ head_project_kernel(const TI* __restrict__ in, long long in_st, long long in_sh,
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int c = j0 + tx * 4 + j;
-            if (c < n_out) out[(long long)t * out_st + h * out_sh + c] = from_float<TO>(acc[i][j]);
+            if (c >= n_out) continue;
+            float v = acc[i][j];
+            if (gate != nullptr) v /= 1.0f + expf(-gate[t * gate_st + (long long)h * n_out + c]);
+            out[(long long)t * out_st + h * out_sh + c] = from_float<TO>(v);
         }
     }
 }
@@ -145,7 +149,7 @@ extern "C" int mlc_latent_prepare(const float* proj, long long stride, const flo
                                   void* k_pool, const int* page_table, long long entry_offset, int pages_per_seq,
                                   int page_size, void* stream) {
     if (n <= 0) return 0;
-    if (H <= 0 || dim < 0 || rot < 0 || (rot & 1) || rank <= 0 || D < rank + rot) return MLC_ERR_BAD_SIZE;
+    if (H <= 0 || dim < 0 || rot < 0 || (rot & 1) || rank <= 0 || D < rank + rot || (write_cache && gain == nullptr)) return MLC_ERR_BAD_SIZE;
     PagedKV c{k_pool, k_pool, page_table, entry_offset, pages_per_seq, page_size, 1, D};
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = 32 * (H + 1 < 8 ? H + 1 : 8);
@@ -165,7 +169,8 @@ extern "C" int mlc_latent_prepare(const float* proj, long long stride, const flo
 
 extern "C" int mlc_head_project(const void* in, int in_dtype, long long in_st, long long in_sh, const void* w, int w_dtype,
                                 long long w_sh, long long w_sd, long long w_sj, void* out, int out_dtype, long long out_st,
-                                long long out_sh, int n, int H, int n_in, int n_out, void* stream) {
+                                long long out_sh, int n, int H, int n_in, int n_out, const float* gate, long long gate_st,
+                                void* stream) {
     if (n <= 0) return 0;
     if (H <= 0 || H > 65535 || n_in <= 0 || n_out <= 0) return MLC_ERR_BAD_SIZE;
     const dim3 grid((n_out + HP_TILE - 1) / HP_TILE, (n + HP_TILE - 1) / HP_TILE, H);
@@ -174,7 +179,7 @@ extern "C" int mlc_head_project(const void* in, int in_dtype, long long in_st, l
     const int code = in_dtype * 4 + w_dtype * 2 + out_dtype;
 #define MLC_HP(TI, TW, TO)                                                                                                  \
     head_project_kernel<TI, TW, TO><<<grid, 256, 0, s>>>((const TI*)in, in_st, in_sh, (const TW*)w, w_sh, w_sd, w_sj, (TO*)out, \
-                                                         out_st, out_sh, n, n_in, n_out)
+                                                         out_st, out_sh, n, n_in, n_out, gate, gate_st)
     switch (code) {
         case 0: MLC_HP(float, float, float); break;
         case 1: MLC_HP(float, float, bf16); break;

@@ -130,19 +130,20 @@ moe_route_kernel(const TX* __restrict__ x, const float* __restrict__ w, const fl
     if (lane < top) weights[(long long)t * top + lane] = p / sum;
 }
 
-// Routing by scores of all experts.  s = softmax(z) over all E router outputs; an expert is *chosen* by s + correction
-// (a stored per-expert term that steers the choice only) and *weighted* by s itself:
-//   groups   the E outputs form G equal groups of neighbours; a group's score is its largest choice score, and only
-//            experts of the `keep` best groups can be chosen (the others count as minus infinity);
+// Routing by scores of all experts.  s = softmax(z) over all E router outputs (SIGMOID: s = sigmoid(z), each on its own); an
+// expert is *chosen* by s + correction (a stored per-expert term that steers the choice only) and *weighted* by s itself:
+//   groups   the E outputs form G equal groups of neighbours; a group's score is its largest choice score (`pair_groups`: the
+//            sum of its two largest), and only experts of the `keep` best groups can be chosen (the others count as minus
+//            infinity);
 //   choice   the `top` largest remaining choice scores (the lower index wins a tie);
 //   weights  s of the chosen, divided by their sum + 1e-20, times `scale`.
 // The last E - n_real outputs belong to identity experts (no matrices: the token's input itself); they are chosen and
 // weighted like the others, and whoever sums the rows treats their ids apart.  A block of four warps per token forms the
 // logits, warp 0 chooses.
-template <typename TX, int PL>
+template <typename TX, int PL, bool SIGMOID>
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const TX* __restrict__ x, const float* __restrict__ w, const float* __restrict__ correction, int n,
-                        int E, int K, int top, int G, int keep, float scale, int* __restrict__ ids,
+                        int E, int K, int top, int G, int keep, int pair_groups, float scale, int* __restrict__ ids,
                         float* __restrict__ weights) {
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -160,18 +161,24 @@ moe_route_scored_kernel(const TX* __restrict__ x, const float* __restrict__ w, c
         z[k] = e < E ? logit[e] : -INFINITY;
         m = fmaxf(m, z[k]);
     }
-    m = warp_max(m);
-    float sum = 0.0f;
+    float sum = 1.0f;
+    if constexpr (SIGMOID) {
 #pragma unroll
-    for (int k = 0; k < PL; ++k) {
-        z[k] = lane + 32 * k < E ? expf(z[k] - m) : 0.0f;
-        sum += z[k];
+        for (int k = 0; k < PL; ++k) z[k] = 1.0f / (1.0f + expf(-z[k]));
+    } else {
+        m = warp_max(m);
+        sum = 0.0f;
+#pragma unroll
+        for (int k = 0; k < PL; ++k) {
+            z[k] = lane + 32 * k < E ? expf(z[k] - m) : 0.0f;
+            sum += z[k];
+        }
+        sum = warp_sum(sum);
     }
-    sum = warp_sum(sum);
 #pragma unroll
     for (int k = 0; k < PL; ++k) {
         const int e = lane + 32 * k;
-        z[k] = z[k] / sum;                            // the score s
+        if constexpr (!SIGMOID) z[k] = z[k] / sum;    // the score s
         c[k] = e < E ? z[k] + (correction != nullptr ? correction[e] : 0.0f) : -INFINITY;
         if (e < E) {
             prob[e] = z[k];
@@ -182,9 +189,13 @@ moe_route_scored_kernel(const TX* __restrict__ x, const float* __restrict__ w, c
     if (G > 1 && keep < G) {
         const int gs = E / G;
         for (int g = lane; g < G; g += 32) {
-            float best = -INFINITY;
-            for (int j = 0; j < gs; ++j) best = fmaxf(best, logit[g * gs + j]);
-            gscore[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int j = 0; j < gs; ++j) {
+                const float v = logit[g * gs + j];
+                second = fmaxf(second, fminf(best, v));
+                best = fmaxf(best, v);
+            }
+            gscore[g] = pair_groups && gs > 1 ? best + second : best;
         }
         __syncwarp();
         // the `keep` best groups, one a round (the lower index wins a tie); a kept group's score is replaced by +infinity
@@ -446,7 +457,8 @@ __global__ void scaled_add_kernel(float* __restrict__ x, const float* __restrict
 }
 
 // x[t][i] += s1[i] · sum_slices y1[.][t][i] + s2[i] · sum_j weights[t][j] · rows[row_of[t][j]][i]: the block's addition with
-// the weighted sum of a token's expert rows made on the way (j in the order of the choices; float32).
+// the weighted sum of a token's expert rows made on the way (j in the order of the choices; float32).  Without y1 (null,
+// slices1 = 0) only the experts' sum is added.
 template <int VEC>
 __global__ void scaled_add_experts_kernel(float* __restrict__ x, const float* __restrict__ y1, int slices1, const float* __restrict__ s1,
                                           const float* __restrict__ rows, const int* __restrict__ row_of,
@@ -497,19 +509,26 @@ extern "C" int mlc_moe_route(const void* x, int x_dtype, const float* w, const f
 }
 
 // x: the branch's input [n][K] of x_dtype; w float32 [E][K]; correction float32 [E] or null.  G groups of which `keep` stay
-// (G <= 1 or keep >= G: no grouping; E must be a multiple of G).
+// (G <= 1 or keep >= G: no grouping; E must be a multiple of G).  sigmoid, pair_groups: see the kernel.
 extern "C" int mlc_moe_route_scored(const void* x, int x_dtype, const float* w, const float* correction, int n, int E, int K,
-                                    int top, int G, int keep, float scale, int* ids, float* weights, void* stream) {
+                                    int top, int G, int keep, int sigmoid, int pair_groups, float scale, int* ids,
+                                    float* weights, void* stream) {
     if (n <= 0) return 0;
     if (E <= 0 || E > 32 * ROUTE_MAX_PER_LANE || top <= 0 || top > 32 || top > E || K <= 0 || w == nullptr) return MLC_ERR_BAD_SIZE;
     if (G > 1 && (E % G != 0 || keep < 1)) return MLC_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
-    if (x_dtype == MLC_DTYPE_F32)
-        (E <= 32 ? moe_route_scored_kernel<float, 1> : moe_route_scored_kernel<float, ROUTE_MAX_PER_LANE>)<<<n, 128, 0, s>>>((const float*)x, w, correction, n, E, K, top, G, keep, scale, ids, weights);
-    else if (x_dtype == MLC_DTYPE_BF16)
-        (E <= 32 ? moe_route_scored_kernel<bf16, 1> : moe_route_scored_kernel<bf16, ROUTE_MAX_PER_LANE>)<<<n, 128, 0, s>>>((const bf16*)x, w, correction, n, E, K, top, G, keep, scale, ids, weights);
-    else
+#define MLC_ROUTE(TX, PL, SG) \
+    moe_route_scored_kernel<TX, PL, SG><<<n, 128, 0, s>>>((const TX*)x, w, correction, n, E, K, top, G, keep, pair_groups, scale, ids, weights)
+#define MLC_ROUTE_SIZES(TX, SG) do { if (E <= 32) MLC_ROUTE(TX, 1, SG); else MLC_ROUTE(TX, ROUTE_MAX_PER_LANE, SG); } while (0)
+    if (x_dtype == MLC_DTYPE_F32) {
+        if (sigmoid) MLC_ROUTE_SIZES(float, true); else MLC_ROUTE_SIZES(float, false);
+    } else if (x_dtype == MLC_DTYPE_BF16) {
+        if (sigmoid) MLC_ROUTE_SIZES(bf16, true); else MLC_ROUTE_SIZES(bf16, false);
+    } else {
         return MLC_ERR_BAD_DTYPE;
+    }
+#undef MLC_ROUTE_SIZES
+#undef MLC_ROUTE
     MLC_LAUNCH_CHECK();
     return 0;
 }
@@ -602,7 +621,7 @@ extern "C" int mlc_scaled_add_experts(float* x, const float* y1, int slices1, co
                                       const int* row_of, const float* weights, int top, const float* s2, long long n, int d,
                                       void* stream) {
     if (n <= 0) return 0;
-    if (d <= 0 || y1 == nullptr || slices1 < 1 || top < 1) return MLC_ERR_BAD_SIZE;
+    if (d <= 0 || (y1 == nullptr ? slices1 != 0 : slices1 < 1) || top < 1) return MLC_ERR_BAD_SIZE;
     const long long total = n * d;
     if ((d & 3) == 0)
         scaled_add_experts_kernel<4><<<(unsigned)((total / 4 + 255) / 256), 256, 0, (cudaStream_t)stream>>>(

@@ -5,7 +5,7 @@ import ctypes
 import functools
 from ctypes import c_float, c_int, c_longlong, c_ulonglong, c_void_p
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -94,8 +94,8 @@ def core() -> ctypes.CDLL:
             "mlc_embed": [P, I, P, I, I, F, P, P],
             "mlc_add_rmsnorm": [P, P, I, P, F, I, I, P, I, P],
             "mlc_rope_table": [P, I, I, F, P, P],
-            "mlc_layernorm": [P, P, I, P, F, I, I, I, P, I, P],
-            "mlc_qk_norm_rope_cache": [P, LL, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P, P, LL, I, I, I, P, P, P, I, I, P],
+            "mlc_layernorm": [P, P, I, P, P, P, I, P, P, F, I, I, I, P, I, P],
+            "mlc_qk_norm_rope_cache": [P, LL, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P, P, LL, I, I, I, P, P, P, I, I, F, I, P],
             "mlc_softcap": [P, LL, F, P],
             "mlc_causal_conv": [P, LL, P, P, P, I, I, I, P, LL, P, P, P, I, I, I, P, LL, P],
             "mlc_gated_delta_rule": [P, LL, I, I, I, P, LL, I, I, P, P, P, P, LL, P, P, I, I, I, I, I, I, I, P, P],
@@ -113,7 +113,7 @@ def core() -> ctypes.CDLL:
             "mlc_grouped_linear": [P, I, P, P, I, P, I, I, I, I, P, I, P],
             "mlc_moe_gather": [P, I, P, I, I, P, P, P, I, P],
             "mlc_moe_combine": [P, P, P, P, I, I, I, I, P, P],
-            "mlc_moe_route_scored": [P, I, P, P, I, I, I, I, I, I, F, P, P, P],
+            "mlc_moe_route_scored": [P, I, P, P, I, I, I, I, I, I, I, I, F, P, P, P],
             "mlc_group_norm": [P, LL, I, I, I, P, I, F, F, P, I, P, P, P, I, P, I, P, LL, P, I, P, I, P],
             "mlc_activation": [P, I, LL, I, P, I, P],
             "mlc_tanh_norm": [P, P, I, P, P, I, P, P, F, F, P, P, F, I, I, P, I, P],
@@ -125,7 +125,7 @@ def core() -> ctypes.CDLL:
             "mlc_scaled_add_experts": [P, P, I, P, P, P, P, I, P, LL, I, P],
             "mlc_gla": [P, LL, I, I, I, P, P, F, P, LL, P, P, I, I, I, I, I, I, P, P],
             "mlc_latent_prepare": [P, LL, P, LL, I, I, I, P, F, P, P, P, I, I, I, I, I, I, I, P, I, I, P, P, LL, I, I, P],
-            "mlc_head_project": [P, I, LL, LL, P, I, LL, LL, LL, P, I, LL, LL, I, I, I, I, P],
+            "mlc_head_project": [P, I, LL, LL, P, I, LL, LL, LL, P, I, LL, LL, I, I, I, I, P, LL, P],
             "mlc_linear_simt": [P, I, P, I, P, I, I, I, I, P, LL, I, P],
             "mlc_attention_combine": [P, P, LL, I, I, P, I, P, I, P],
             "mlc_gemm_tcgen05": [P, P, P, I, I, I, I, I, I, I, P, P, I, P, P, P, P, I, I, I, I, P, P, P, LL, I, I, I, F, F, P],
@@ -371,21 +371,36 @@ def decode_advance(chosen: torch.Tensor, tokens: torch.Tensor, positions: torch.
 
 
 
+def _expert_rows(expert_rows, n: int, d: int):
+    """(rows, row_of, weights, top) of a token's expert rows as a kernel's branch, checked; Nones and 0 without them."""
+    if expert_rows is None:
+        return None, None, None, 0
+    rows, row_of, weights = expert_rows
+    require_cuda(rows, row_of, weights)
+    assert rows.dtype == weights.dtype == torch.float32 and row_of.dtype == torch.int32 and rows.shape[1] == d
+    assert row_of.shape == weights.shape and row_of.shape[0] == n
+    return rows, row_of, weights, row_of.shape[1]
+
+
 def layernorm(x: torch.Tensor, y: Optional[torch.Tensor], gain: torch.Tensor, eps: float, out: Optional[torch.Tensor],
-              of_branch: bool) -> None:
-    """Layer norm with a gain and no bias, statistics in float32.  `of_branch` False: x (float32 [n, d]) += y if given
-    ([n, d] or slices [s, n, d] that are added up), out = LN(x).  `of_branch` True: x += LN(y); out, if given, receives
-    the new x in its own type."""
-    require_cuda(x, y, gain, out)
+              of_branch: bool, bias: Optional[torch.Tensor] = None, expert_rows=None) -> None:
+    """Layer norm with a gain and an optional bias, statistics in float32.  The branch is y ([n, d] or slices [s, n, d] that
+    are added up) or `expert_rows` = (rows float32 [., d], row_of int32 [n, top], weights float32 [n, top]), the weighted sum
+    of each token's expert rows.  `of_branch` False: x (float32 [n, d]) += branch if given, out = LN(x).  `of_branch` True:
+    x += LN(branch); out, if given, receives the new x in its own type."""
+    require_cuda(x, y, gain, out, bias)
     n, d = x.shape
     assert x.dtype == torch.float32 and gain.dtype == torch.float32 and gain.numel() == d
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == d)
     assert out is None or out.shape == x.shape
+    rows, row_of, weights, top = _expert_rows(expert_rows, n, d)
     n_slices = 1
     if y is not None:
         assert y.dtype == torch.float32 and tuple(y.shape[-2:]) == (n, d)
         n_slices = y.shape[0] if y.dim() == 3 else 1
-    _check(core().mlc_layernorm(x.data_ptr(), _ptr(y), n_slices, gain.data_ptr(), float(eps), n, d, 1 if of_branch else 0,
-                                _ptr(out), dtype_code(out.dtype) if out is not None else 0, _stream()), "layer norm")
+    _check(core().mlc_layernorm(x.data_ptr(), _ptr(y), n_slices, _ptr(rows), _ptr(row_of), _ptr(weights), top,
+                                gain.data_ptr(), _ptr(bias), float(eps), n, d, 1 if of_branch else 0, _ptr(out),
+                                dtype_code(out.dtype) if out is not None else 0, _stream()), "layer norm")
 
 
 def qk_norm_rope_cache(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_gain: Optional[torch.Tensor],
@@ -393,13 +408,16 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
                        rope: Optional[torch.Tensor], rot_dims: int, q_heads: int, kv_heads_in_row: int, dim: int, vdim: int,
                        v_scale: float, q_out: torch.Tensor, kv: Optional[KVView], q_bias: Optional[torch.Tensor] = None,
                        k_bias: Optional[torch.Tensor] = None, v_bias: Optional[torch.Tensor] = None, whole_row: bool = False,
-                       interleaved: bool = False) -> None:
+                       interleaved: bool = False, q_temp: Optional[Tuple[float, int]] = None) -> None:
     """Rows of a float32 projection (q heads at column q_col, k heads at k_col, v heads at v_col): per-head RMS norm of q
     and k (gain optional; a negative eps: none), rotation of the first `rot_dims` entries of each head by the table
     `rope` [positions, rot_dims/2, 2], v times `v_scale`; q into q_out [n, q_heads, D], k and v into the cache, whose
     heads have D >= max(dim, vdim) entries (the rest zero).  Biases (float32, as long as their projections) are added as the
     columns are read.  `whole_row`: one statistic over all q heads and one over all k heads, gains as long as the
-    projections.  `interleaved`: the rotation pairs entry 2j with 2j + 1 instead of j with j + rot_dims/2."""
+    projections.  `interleaved`: the rotation pairs entry 2j with 2j + 1 instead of j with j + rot_dims/2.  `q_temp` =
+    (coef, every): the queries of position p are multiplied by 1 + coef · ln(floor((p + 1) / every) + 1)."""
+    coef, every = q_temp if q_temp is not None else (0.0, 0)
+    assert every >= 0
     require_cuda(proj, q_gain, k_gain, positions, tok_seq, rope, q_out, q_bias, k_bias, v_bias)
     for g, heads in ((q_gain, q_heads), (k_gain, kv_heads_in_row)):
         assert g is None or not heads or g.numel() == (heads * dim if whole_row else dim)
@@ -421,7 +439,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
                                          rope.shape[0] if rope is not None else 0, rot_dims if rope is not None else 0, n,
                                          q_heads, kv_heads_in_row, dim, vdim, D, float(v_scale), q_out.data_ptr(),
                                          dtype_code(q_out.dtype), *args, _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
-                                         1 if whole_row else 0, 1 if interleaved else 0, _stream()),
+                                         1 if whole_row else 0, 1 if interleaved else 0, float(coef), int(every), _stream()),
            "q/k norm, rotation and cache write")
 
 
@@ -647,11 +665,12 @@ def moe_combine(y: torch.Tensor, row_of: torch.Tensor, weights: Optional[torch.T
 
 
 def moe_route_scored(x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int,
-                     scale: float, ids: torch.Tensor, weights: torch.Tensor) -> None:
-    """Routing by the softmax s over all router outputs (router float32 [E, K], x the branch's input [n, K]; logits in
-    float32): chosen are the `top` largest s + correction among the experts of the `keep` best of `groups` equal groups of
-    neighbours (a group's score: its largest choice score; groups <= 1: no grouping); weights = s of the chosen, divided
-    by their sum + 1e-20, times `scale`.  ids int32 [n, top], weights float32 [n, top]."""
+                     scale: float, ids: torch.Tensor, weights: torch.Tensor, score: str = "softmax", group_score: str = "max") -> None:
+    """Routing by scores s of all router outputs (router float32 [E, K], x the branch's input [n, K]; logits in float32;
+    `score`: s is the "softmax" over all outputs, or each output's own "sigmoid"): chosen are the `top` largest
+    s + correction among the experts of the `keep` best of `groups` equal groups of neighbours (a group's score: its largest
+    choice score, "max", or the sum of its two largest, "top2"; groups <= 1: no grouping); weights = s of the chosen,
+    divided by their sum + 1e-20, times `scale`.  ids int32 [n, top], weights float32 [n, top]."""
     require_cuda(x, router, correction, ids, weights)
     n = x.shape[0]
     E, K = router.shape
@@ -659,7 +678,8 @@ def moe_route_scored(x: torch.Tensor, router: torch.Tensor, correction: Optional
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.shape == (n, top) and weights.shape == (n, top)
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
     _check(core().mlc_moe_route_scored(x.data_ptr(), dtype_code(x.dtype), router.data_ptr(), _ptr(correction), n, E, K, int(top),
-                                       int(groups), int(keep), float(scale), ids.data_ptr(), weights.data_ptr(), _stream()),
+                                       int(groups), int(keep), {"softmax": 0, "sigmoid": 1}[score],
+                                       {"max": 0, "top2": 1}[group_score], float(scale), ids.data_ptr(), weights.data_ptr(), _stream()),
            "expert routing by scores")
 
 
@@ -678,17 +698,19 @@ def scaled_add(x: torch.Tensor, y1: torch.Tensor, s1: Optional[torch.Tensor], y2
            "scaled addition")
 
 
-def scaled_add_experts(x: torch.Tensor, y1: torch.Tensor, s1: Optional[torch.Tensor], rows: torch.Tensor, row_of: torch.Tensor,
+def scaled_add_experts(x: torch.Tensor, y1: Optional[torch.Tensor], s1: Optional[torch.Tensor], rows: torch.Tensor, row_of: torch.Tensor,
                        weights: torch.Tensor, s2: Optional[torch.Tensor]) -> None:
     """x (float32 [n, d], in place) += s1 · y1 + s2 · f, where f[t] = sum_j weights[t, j] · rows[row_of[t, j]] is the weighted
-    sum of token t's expert rows (`moe_combine`'s result, made on the way instead of stored)."""
+    sum of token t's expert rows (`moe_combine`'s result, made on the way instead of stored); without y1, s2 · f alone."""
     require_cuda(x, y1, s1, rows, row_of, weights, s2)
     n, d = x.shape
-    assert y1.dtype == rows.dtype == weights.dtype == torch.float32 and tuple(y1.shape[-2:]) == (n, d) and rows.shape[1] == d
+    assert rows.dtype == weights.dtype == torch.float32 and rows.shape[1] == d
+    assert y1 is None or (y1.dtype == torch.float32 and tuple(y1.shape[-2:]) == (n, d))
+    slices = 0 if y1 is None else y1.shape[0] if y1.dim() == 3 else 1
     assert row_of.dtype == torch.int32 and row_of.shape == weights.shape and row_of.shape[0] == n
     for f in (s1, s2):
         assert f is None or (f.dtype == torch.float32 and f.numel() == d)
-    _check(core().mlc_scaled_add_experts(x.data_ptr(), y1.data_ptr(), y1.shape[0] if y1.dim() == 3 else 1, _ptr(s1), rows.data_ptr(),
+    _check(core().mlc_scaled_add_experts(x.data_ptr(), _ptr(y1), slices, _ptr(s1), rows.data_ptr(),
                                          row_of.data_ptr(), weights.data_ptr(), row_of.shape[1], _ptr(s2), n, d, _stream()),
            "scaled addition of expert rows")
 
@@ -884,7 +906,7 @@ def activation(src: torch.Tensor, kind: str, out: torch.Tensor) -> None:
 
 
 # ------------------------------------------------------------------ latent attention (csrc/latent.cu)
-def latent_prepare(proj: torch.Tensor, q_col: int, kv_col: int, gain: torch.Tensor, eps: float, positions: torch.Tensor,
+def latent_prepare(proj: torch.Tensor, q_col: int, kv_col: int, gain: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
                    tok_seq: torch.Tensor, rope: Optional[torch.Tensor], heads: int, dim: int, rot: int, rank: int,
                    q_out: torch.Tensor, kv: Optional[KVView], q_rows: Optional[torch.Tensor] = None,
                    interleaved: bool = False) -> None:
@@ -892,13 +914,14 @@ def latent_prepare(proj: torch.Tensor, q_col: int, kv_col: int, gain: torch.Tens
     [normed latent | rotated shared key part | zeros] of every token (when `kv` is given), and the rotated query parts
     into entries [rank, rank + rot) of q_out [n, heads, D] (zeros behind them).  With `q_rows` (float32 rows) the query
     heads are read from there instead, at q_col.  `interleaved`: the rotation pairs entry 2i with 2i + 1, not i with
-    i + rot/2."""
+    i + rot/2.  Without `kv` (the latent belongs to another run) the gain may be absent and kv_col is not read."""
     require_cuda(proj, gain, positions, tok_seq, rope, q_out)
     qsrc = proj if q_rows is None else q_rows
     assert qsrc.dtype == torch.float32 and qsrc.dim() == 2 and qsrc.stride(1) == 1 and qsrc.shape[0] == proj.shape[0]
     n = proj.shape[0]
     D = q_out.numel() // max(1, n * heads)
-    assert proj.dtype == torch.float32 and gain.dtype == torch.float32 and gain.numel() == rank
+    assert proj.dtype == torch.float32 and (gain is not None or kv is None)
+    assert gain is None or (gain.dtype == torch.float32 and gain.numel() == rank)
     assert rope is None or (rope.dtype == torch.float32 and rope.shape[1] * 2 == rot)
     if kv is not None:
         assert kv.k_pool.dtype == q_out.dtype and kv.head_dim == D and kv.kv_heads == 1
@@ -906,22 +929,25 @@ def latent_prepare(proj: torch.Tensor, q_col: int, kv_col: int, gain: torch.Tens
     else:
         args = (0, None, None, 0, 0, 1)
     _check(core().mlc_latent_prepare(proj.data_ptr(), proj.stride(0), qsrc.data_ptr(), qsrc.stride(0), 1 if interleaved else 0,
-                                     q_col, kv_col, gain.data_ptr(), float(eps),
+                                     q_col, kv_col, _ptr(gain), float(eps),
                                      positions.data_ptr(), tok_seq.data_ptr(), _ptr(rope), rope.shape[0] if rope is not None else 0,
                                      n, heads, dim, rot, rank, D, q_out.data_ptr(), dtype_code(q_out.dtype), *args, _stream()),
            "latent norm, rotation and cache write")
 
 
 def head_project(src: torch.Tensor, src_strides, w: torch.Tensor, w_strides, out: torch.Tensor, out_strides, n: int, heads: int,
-                 n_in: int, n_out: int, src_offset: int = 0, out_offset: int = 0) -> None:
+                 n_in: int, n_out: int, src_offset: int = 0, out_offset: int = 0, gate: Optional[torch.Tensor] = None,
+                 gate_col: int = 0) -> None:
     """out[t, h, j] = sum_d src[t, h, d] · w[h, d, j] per head with float32 multiply-adds.  Strides in elements:
-    src (token, head), w (head, d, j), out (token, head); offsets in elements from each tensor's start."""
+    src (token, head), w (head, d, j), out (token, head); offsets in elements from each tensor's start.  With `gate`
+    (float32 rows) out[t, h, j] is multiplied by sigmoid(gate[t, gate_col + h · n_out + j]) before it is rounded."""
     require_cuda(src, w, out)
     lib = core()
     _check(lib.mlc_head_project(src.data_ptr() + src_offset * src.element_size(), dtype_code(src.dtype), src_strides[0], src_strides[1],
                                 w.data_ptr(), dtype_code(w.dtype), w_strides[0], w_strides[1], w_strides[2],
                                 out.data_ptr() + out_offset * out.element_size(), dtype_code(out.dtype), out_strides[0], out_strides[1],
-                                n, heads, n_in, n_out, _stream()), "per-head product")
+                                n, heads, n_in, n_out, _columns(gate, gate_col) if gate is not None else None,
+                                gate.stride(0) if gate is not None else 0, _stream()), "per-head product")
 
 
 class PinnedCopy:

@@ -13,7 +13,7 @@ all sequences, run at once against the cache.
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -152,7 +152,11 @@ class GQAttention(Part):
                              memory.kv if memory.writes_cache else None)
         o = rt.empty(n, self.H * self.hd)
         self.attend(q, o, step, memory.kv)
-        if residual is not None and self.o.can_add_into_stream(n):
+        return self._out(o, residual)
+
+    def _out(self, o: torch.Tensor, residual: Optional[torch.Tensor]):
+        """The output product: added into the stream `residual` if that is given and its product can (returns None)."""
+        if residual is not None and self.o.can_add_into_stream(o.shape[0]):
             self.o.add_into(o, residual)
             return None
         return self.o(o, torch.float32, partial_ok=True)
@@ -242,12 +246,14 @@ class SinkAttention(GQAttention):
     tensors (projections, biases, key norm) and only ever reads another run's cache entry, with queries, mask and everything
     else of its own.  `keep_all_keys`: the cache keeps every position whatever this mixer's own mask (for an entry that
     another run reads under another mask).  The position part's `interleaved` says which entries form a rotation pair.
+    `qk_gain=False`: the norm of queries and keys has no gain (no q_norm and k_norm tensors).  `const_sink`: instead of a
+    learned sink per head, one number for all of them (0: the softmax has one more in its denominator).  `q_temp` =
+    (coef, every): the queries of position p are multiplied by 1 + coef · ln(floor((p + 1) / every) + 1), in float32.
 
     `names`: the tensors' names below the part's prefix, by role (q, k, v, o, q_norm, k_norm, sink, g; a bias is its matrix's
     name with `.b`).  Offers `in_weights()` and `mix()` to an arrangement that computes several mixers' input projections in
     one product."""
     graph_safe = True
-    accumulates = False
 
     NAMES = dict(q="q", k="k", v="v", o="o", q_norm="q.norm", k_norm="k.norm", sink="sink", g="g")
 
@@ -255,12 +261,13 @@ class SinkAttention(GQAttention):
                  scale: float, norm_eps: float, position: PartSpec, qk_norm: bool = True, sink: bool = True,
                  window: Optional[int] = None, value_scale: float = 1.0, names: Optional[dict] = None, keep_first: int = 0,
                  bias: bool = False, softcap: Optional[float] = None, chunk: Optional[int] = None, out_gate: bool = False,
-                 own_kv: bool = True, keep_all_keys: bool = False):
+                 own_kv: bool = True, keep_all_keys: bool = False, qk_gain: bool = True, const_sink: Optional[float] = None,
+                 q_temp: Optional[Tuple[float, int]] = None):
         """`window`, `keep_first`: position i sees j <= i with i - j < window or j < keep_first (no window: every j <= i)."""
         Part.__init__(self, name, hidden_size=hidden_size, num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim,
                       v_head_dim=v_head_dim, scale=scale, norm_eps=norm_eps, qk_norm=qk_norm, sink=sink, window=window,
                       value_scale=value_scale, keep_first=keep_first, bias=bias, softcap=softcap, chunk=chunk, out_gate=out_gate,
-                      own_kv=own_kv, keep_all_keys=keep_all_keys)
+                      own_kv=own_kv, keep_all_keys=keep_all_keys, qk_gain=qk_gain, const_sink=const_sink, q_temp=q_temp)
         if num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} kv heads")
         self.hidden, self.H, self.KV = int(hidden_size), int(num_heads), int(num_kv_heads)
@@ -272,6 +279,13 @@ class SinkAttention(GQAttention):
             raise ValueError(f"attention: the score's scale must be positive, got {scale}")
         self.scale, self.eps = float(scale), float(norm_eps)
         self.qk_norm, self.has_sink = bool(qk_norm), bool(sink)
+        self.qk_gain = self.qk_norm and bool(qk_gain)
+        self.const_sink = float(const_sink) if const_sink is not None else None
+        if self.has_sink and self.const_sink is not None:
+            raise ValueError("attention: a learned sink excludes a constant one")
+        self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else None
+        if self.q_temp is not None and self.q_temp[1] < 1:
+            raise ValueError(f"attention: the query temperature's period must be positive, got {q_temp[1]}")
         self.window = int(window) if window else None
         self.keep_first = max(0, int(keep_first)) if self.window else 0
         self.value_scale = float(value_scale)
@@ -298,7 +312,7 @@ class SinkAttention(GQAttention):
             if self.own_kv:
                 specs += [TensorSpec(t["k"] + ".b", (self.KV * self.dim,), role="bias"),
                           TensorSpec(t["v"] + ".b", (self.KV * self.vdim,), role="bias")]
-        if self.qk_norm:
+        if self.qk_gain:
             specs.append(TensorSpec(t["q_norm"], (self.dim,), role="gain", init="one_plus_normal"))
             if self.own_kv:
                 specs.append(TensorSpec(t["k_norm"], (self.dim,), role="gain", init="one_plus_normal"))
@@ -322,12 +336,14 @@ class SinkAttention(GQAttention):
         # columns of the input product: q | k | v | g (without the parts the mixer does not have)
         self._in = [get(t["q"])] + ([get(t["k"]), get(t["v"])] if self.own_kv else []) + ([get(t["g"])] if self.out_gate else [])
         self.in_proj: Optional[Linear] = None
-        self.q_gain = f32(t["q_norm"]) if self.qk_norm else None
-        self.k_gain = f32(t["k_norm"]) if self.qk_norm and self.own_kv else None
+        self.q_gain = f32(t["q_norm"]) if self.qk_gain else None
+        self.k_gain = f32(t["k_norm"]) if self.qk_gain and self.own_kv else None
         self.q_bias = f32(t["q"] + ".b") if self.has_bias else None
         self.k_bias = f32(t["k"] + ".b") if self.has_bias and self.own_kv else None
         self.v_bias = f32(t["v"] + ".b") if self.has_bias and self.own_kv else None
         self.sinks = f32(t["sink"]) if self.has_sink else None
+        if self.const_sink is not None:
+            self.sinks = torch.full((self.H,), self.const_sink, dtype=torch.float32, device=runtime.device)
         wo = get(t["o"])
         if self.hd != self.vdim:            # the kernels' heads are wider than the values: columns of zeros
             padded = torch.zeros(self.hidden, self.H, self.hd, dtype=wo.dtype, device=wo.device)
@@ -367,7 +383,7 @@ class SinkAttention(GQAttention):
         kernels.qk_norm_rope_cache(proj, q_col, k_col, v_col, self.q_gain, self.k_gain, self.eps if self.qk_norm else -1.0,
                                    step.positions, step.tok_seq, table, rot, self.H, kv_heads, self.dim, self.vdim,
                                    self.value_scale, q, memory.kv if memory.writes_cache else None, q_bias=self.q_bias,
-                                   k_bias=self.k_bias, v_bias=self.v_bias, interleaved=self.interleaved)
+                                   k_bias=self.k_bias, v_bias=self.v_bias, interleaved=self.interleaved, q_temp=self.q_temp)
         o = rt.empty(n, self.H * self.hd)
         self.attend(q, o, step, memory.kv)
         if self.out_gate:
@@ -377,8 +393,7 @@ class SinkAttention(GQAttention):
     def forward(self, h: torch.Tensor, step, memory: MixerMemory, residual: Optional[torch.Tensor] = None):
         if self.in_proj is None:
             self.in_proj = fused_rows(self._in, self.runtime)
-        o = self.mix(self.in_proj(h, torch.float32), 0, step, memory)
-        return self.o(o, torch.float32, partial_ok=True)
+        return self._out(self.mix(self.in_proj(h, torch.float32), 0, step, memory), residual)
 
 
 @register_part("mixer", "latent_attention")
@@ -400,22 +415,28 @@ class LatentAttention(GQAttention):
     Options.  `q_rank`: the queries go through a latent of their own, c_q = rms(W_dq h) · g_q (eps inside the root),
     q = W_uq c_q (tensors dq, dq_norm, uq instead of q).  `window`: position i sees the keys j with 0 <= i - j < window
     (no window: every j <= i); the cache then keeps a window of rows.  The position part's `interleaved` says which
-    entries of the rotated part form a pair.
+    entries of the rotated part form a pair.  `sink`: a learned logit per head (tensor `sink`) that joins the softmax's
+    denominator once, with no key and no value, outside the scale.  `out_gate`: the heads' values are multiplied entry by
+    entry by sigmoid(W_g h) before the output product; W_g (`g`) reads the mixer's input and rides in the input product, and
+    the value expansion's kernel applies the gate in float32.  `own_kv=False`: the mixer has no W_dkv (and no norm of a
+    latent) and reads the latents of another run's cache entry, with queries, expansions, sink and gate of its own.
 
     Offers `in_weights()`, `in_width()`, `mix()` and `o` to an arrangement that computes other matrices on the same input
     in the mixer's input product.
 
-    `names`: the tensors' names below the part's prefix, by role (q, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o)."""
+    `names`: the tensors' names below the part's prefix, by role (q, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o, sink, g)."""
     graph_safe = True
-    accumulates = False
 
-    NAMES = dict(q="q", dq="dq", dq_norm="dq.norm", uq="uq", dkv="dkv", dkv_norm="dkv.norm", uk="uk", uv="uv", o="o")
+    NAMES = dict(q="q", dq="dq", dq_norm="dq.norm", uq="uq", dkv="dkv", dkv_norm="dkv.norm", uk="uk", uv="uv", o="o", sink="sink", g="g")
 
     def __init__(self, name: str, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int,
                  scale: float, norm_eps: float, position: PartSpec, names: Optional[dict] = None, q_rank: Optional[int] = None,
-                 window: Optional[int] = None):
+                 window: Optional[int] = None, sink: bool = False, out_gate: bool = False, own_kv: bool = True):
         Part.__init__(self, name, hidden_size=hidden_size, num_heads=num_heads, head_dim=head_dim, rot_dim=rot_dim,
-                      v_head_dim=v_head_dim, kv_rank=kv_rank, scale=scale, norm_eps=norm_eps, q_rank=q_rank, window=window)
+                      v_head_dim=v_head_dim, kv_rank=kv_rank, scale=scale, norm_eps=norm_eps, q_rank=q_rank, window=window,
+                      sink=sink, out_gate=out_gate, own_kv=own_kv)
+        self.has_sink, self.out_gate, self.own_kv = bool(sink), bool(out_gate), bool(own_kv)
+        self.sinks: Optional[torch.Tensor] = None
         self.hidden, self.H, self.KV = int(hidden_size), int(num_heads), 1
         self.dim, self.rot, self.vdim, self.rank = int(head_dim), int(rot_dim), int(v_head_dim), int(kv_rank)
         self.q_rank = int(q_rank) if q_rank else None
@@ -441,9 +462,14 @@ class LatentAttention(GQAttention):
                  TensorSpec(t["uq"], (nq, self.q_rank))]
         else:
             q = [TensorSpec(t["q"], (nq, self.hidden))]
-        return q + [TensorSpec(t["dkv"], (self.rank + self.rot, self.hidden)),
-                    TensorSpec(t["dkv_norm"], (self.rank,), role="gain", init="one_plus_normal"),
-                    TensorSpec(t["uk"], (H * self.dim, self.rank)), TensorSpec(t["uv"], (H * self.vdim, self.rank)),
+        if self.own_kv:
+            q += [TensorSpec(t["dkv"], (self.rank + self.rot, self.hidden)),
+                  TensorSpec(t["dkv_norm"], (self.rank,), role="gain", init="one_plus_normal")]
+        if self.has_sink:
+            q.append(TensorSpec(t["sink"], (H,), role="bias"))
+        if self.out_gate:
+            q.append(TensorSpec(t["g"], (H * self.vdim, self.hidden)))
+        return q + [TensorSpec(t["uk"], (H * self.dim, self.rank)), TensorSpec(t["uv"], (H * self.vdim, self.rank)),
                     TensorSpec(t["o"], (self.hidden, H * self.vdim))]
 
     def cache_need(self) -> CacheNeed:
@@ -452,15 +478,18 @@ class LatentAttention(GQAttention):
     def bind(self, get, runtime):
         Part.bind(self, get, runtime)
         t = self.t
-        # columns of the input product: [q heads | latent | shared rotated key part], or with a query latent
-        # [query latent | latent | shared rotated key part]
-        self._in = [get(t["dq"]) if self.q_rank else get(t["q"]), get(t["dkv"])]
+        # columns of the input product: [q heads | latent | shared rotated key part | gate], or with a query latent
+        # [query latent | latent | shared rotated key part | gate], without the parts the mixer does not have
+        self._in = ([get(t["dq"]) if self.q_rank else get(t["q"])] + ([get(t["dkv"])] if self.own_kv else [])
+                    + ([get(t["g"])] if self.out_gate else []))
         self.in_proj: Optional[Linear] = None
         self.kv_col = self._in[0].shape[0]
+        self.gate_col = self.kv_col + (self.rank + self.rot if self.own_kv else 0)
+        self.sinks = get(t["sink"]).to(torch.float32).contiguous() if self.has_sink else None
         if self.q_rank:
             self.q_gain = get(t["dq_norm"]).to(torch.float32).contiguous()
             self.uq = Linear(get(t["uq"]), runtime)
-        self.gain = get(t["dkv_norm"]).to(torch.float32).contiguous()
+        self.gain = get(t["dkv_norm"]).to(torch.float32).contiguous() if self.own_kv else None
         self.w_uk, self.w_uv = get(t["uk"]).contiguous(), get(t["uv"]).contiguous()
         self.o = Linear(get(t["o"]), runtime)
         # rows of more than 256 entries run on the float32-arithmetic kernel in both engine types (the tensor-core
@@ -474,7 +503,7 @@ class LatentAttention(GQAttention):
         return list(self._in)
 
     def in_width(self) -> int:
-        return self.kv_col + self.rank + self.rot
+        return sum(w.shape[0] for w in self._in)
 
     def weight_bytes(self) -> int:
         b = sum(w.numel() * w.element_size() for w in self._in) + self.o.nbytes()
@@ -491,6 +520,9 @@ class LatentAttention(GQAttention):
         returns the heads' values [n, heads·vdim] in the engine's type, the input of `self.o`."""
         rt = self.runtime
         n, H, D = proj.shape[0], self.H, self.hd
+        if memory.writes_cache != self.own_kv:
+            raise ValueError("latent attention: a mixer without a latent of its own reads another run's cache entry, and only "
+                             "such a mixer does")
         q_rows, q_col = None, col
         if self.q_rank:
             cq = rt.empty(n, self.q_rank)
@@ -513,14 +545,13 @@ class LatentAttention(GQAttention):
         # the value expansion behind the sum: val[t, h] = W_uv,h (sum_j p c_j)
         val = rt.empty(n, H * self.vdim)
         kernels.head_project(o, (H * D, D), self.w_uv, (self.vdim * self.rank, 1, self.rank), val, (H * self.vdim, self.vdim),
-                             n, H, self.rank, self.vdim)
+                             n, H, self.rank, self.vdim, gate=proj if self.out_gate else None, gate_col=col + self.gate_col)
         return val
 
     def forward(self, h: torch.Tensor, step, memory: MixerMemory, residual: Optional[torch.Tensor] = None):
         if self.in_proj is None:
             self.in_proj = fused_rows(self._in, self.runtime)
-        val = self.mix(self.in_proj(h, torch.float32), 0, step, memory)
-        return self.o(val, torch.float32, partial_ok=True)
+        return self._out(self.mix(self.in_proj(h, torch.float32), 0, step, memory), residual)
 
 
 @register_part("mixer", "conv_attention")
@@ -538,7 +569,6 @@ class ConvKeyAttention(SinkAttention):
     `interleaved` says which entries form a rotation pair.  `names`: the tensors' names below the part's prefix, by role
     (q, k, o, q_norm, k_norm, q_conv, k_conv)."""
     graph_safe = True
-    accumulates = False
 
     NAMES = dict(q="q", k="k", o="o", q_norm="q.norm", k_norm="k.norm", q_conv="q.conv", k_conv="k.conv")
 

@@ -4,7 +4,8 @@ Pre-norm: x ← x + mixer(norm(x)); x ← x + feed_forward(norm(x)) (src/forward
 The additions are deferred: a branch's output travels as `pending` and is added, in
 float32, by the next norm's kernel — the block's own second norm, the next block's first
 norm, or the model's final norm.  On the tensor-core path of small steps the addition moves into
-the preceding product's epilogue (atomic adds into the stream) and nothing is pending at all."""
+the preceding product's epilogue (atomic adds into the stream) and nothing is pending at all.
+A mixture of experts leaves its weighted sum to the next norm's kernel in the same way (`DeferredBranch`)."""
 from __future__ import annotations
 
 from typing import Optional, Tuple
@@ -19,28 +20,47 @@ from .base import MixerMemory, Part, TensorSpec
 
 @register_part("block", "prenorm")
 class PreNormBlock(Part):
+    """The feed-forward (with its norm) may be absent."""
     graph_safe = True
+    takes_deferred_update = True
 
-    def __init__(self, name: str, mixer: PartSpec, feed_forward: PartSpec, mixer_norm: PartSpec,
-                 feed_forward_norm: PartSpec, names: Optional[dict] = None):
+    def __init__(self, name: str, mixer: PartSpec, mixer_norm: PartSpec, feed_forward: Optional[PartSpec] = None,
+                 feed_forward_norm: Optional[PartSpec] = None, names: Optional[dict] = None):
         super().__init__(name)
         names = names or {}
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("prenorm block: a feed-forward and its norm come together or not at all")
         self.mixer_norm = build_part(mixer_norm, name + names.get("mixer_norm", "mixer_norm."))
         self.mixer = build_part(mixer, name + names.get("mixer", "mixer."))
-        self.feed_forward_norm = build_part(feed_forward_norm, name + names.get("feed_forward_norm", "feed_forward_norm."))
-        self.feed_forward = build_part(feed_forward, name + names.get("feed_forward", "feed_forward."))
+        self.feed_forward_norm = (build_part(feed_forward_norm, name + names.get("feed_forward_norm", "feed_forward_norm."))
+                                  if feed_forward_norm else None)
+        self.feed_forward = build_part(feed_forward, name + names.get("feed_forward", "feed_forward.")) if feed_forward else None
 
     def children(self):
-        return (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None)
 
     def forward(self, x: torch.Tensor, pending: Optional[torch.Tensor], step, memory: MixerMemory
                 ) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         """A part either adds its output into the stream x itself (`accumulates`, asked through `residual=x`;
-        it then returns None) or returns its output, which waits in `pending` for the next norm to add it."""
+        it then returns None) or returns its output, which waits in `pending` for the next norm to add it.  A mixture of
+        experts that defers its sum leaves its rows in the step's `handover`, for the next block's first norm (if that
+        norm takes expert rows) or for whoever else reads the stream next."""
         mixer, ffn = self.mixer, self.feed_forward
-        h = self.mixer_norm.forward(x, pending)
+        left = step.handover.pop(DEFERRED, None) if step.handover else None
+        if (left is not None and left.x is x and left.norm is None and left.expert_rows is not None and pending is None
+                and getattr(self.mixer_norm, "takes_expert_rows", False)):
+            h = self.mixer_norm.forward(x, expert_rows=left.expert_rows)
+        else:
+            if left is not None:
+                left.finish()
+            h = self.mixer_norm.forward(x, pending)
         a = mixer.forward(h, step, memory, residual=x) if getattr(mixer, "accumulates", False) else mixer.forward(h, step, memory)
+        if ffn is None:
+            return x, a
         h2 = self.feed_forward_norm.forward(x, a)
+        if getattr(ffn, "defers_sum", False) and not getattr(ffn, "identity", 0) and not getattr(ffn, "sum_is_plain", False):
+            step.handover[DEFERRED] = DeferredBranch(x, expert_rows=ffn.forward(h2, step, deferred=True))
+            return x, None
         f = ffn.forward(h2, step, residual=x) if getattr(ffn, "accumulates", False) else ffn.forward(h2, step)
         return x, f
 
@@ -316,13 +336,17 @@ class StreamMix(Part):
 
 
 class DeferredBranch:
-    """A branch output that a block left for whoever reads the stream next: x += mult · norm(branch) is still to be done.
-    The next block of the same kind does it inside its own first norm's kernel; anybody else calls `finish()`."""
+    """A branch output that a block left for whoever reads the stream next: x += mult · norm(branch) is still to be done, or,
+    without a norm, x += the weighted sum of `expert_rows` = (rows, row_of, weights).  The next block of the same kind does it
+    inside its own first norm's kernel; anybody else calls `finish()`."""
 
-    def __init__(self, x: torch.Tensor, norm, mult: float, y: Optional[torch.Tensor] = None, expert_rows=None):
+    def __init__(self, x: torch.Tensor, norm=None, mult: float = 1.0, y: Optional[torch.Tensor] = None, expert_rows=None):
         self.x, self.norm, self.mult, self.y, self.expert_rows = x, norm, mult, y, expert_rows
 
     def finish(self) -> None:
+        if self.norm is None:
+            kernels.scaled_add_experts(self.x, None, None, *self.expert_rows, None)
+            return
         self.norm.add_normed(self.x, y=self.y, expert_rows=self.expert_rows, mult=self.mult)
 
 
@@ -374,7 +398,7 @@ class SandwichBlock(Part):
     def forward(self, x: torch.Tensor, pending: Optional[torch.Tensor], step, memory: MixerMemory
                 ) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         left = step.handover.pop(DEFERRED, None)
-        if left is not None and left.x is x and pending is None:
+        if left is not None and left.norm is not None and left.x is x and pending is None:
             # the block before left its last addition: it and this block's first norm are one kernel
             h = left.norm.add_normed(x, y=left.y, expert_rows=left.expert_rows, mult=left.mult, then=self.mixer_norm)
         else:

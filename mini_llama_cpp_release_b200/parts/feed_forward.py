@@ -85,10 +85,11 @@ class MixtureOfExperts(Part):
 
     Routing, `routing="top_logits"`: router logits z = W_r h + b_r in float32; each token uses the `top` experts with the
     largest logits, weighted by the softmax over those chosen logits only.  `routing="scores"`: s = softmax(z) over all
-    router outputs; chosen are the `top` largest s + correction (a stored per-expert term, `correction=True`) among the
-    experts of the `group_keep` best of `group_count` equal groups of neighbours (a group's score is its largest choice
-    score; one group: no grouping); the weights are s of the chosen (without the correction), divided by their sum
-    + 1e-20, times `weight_scale`.  `identity`: that many further router outputs, behind the experts', belong to identity
+    router outputs, or with `score="sigmoid"` each output's own sigmoid; chosen are the `top` largest s + correction (a
+    stored per-expert term, `correction=True`) among the experts of the `group_keep` best of `group_count` equal groups of
+    neighbours (a group's score is its largest choice score, `group_score="max"`, or the sum of its two largest, "top2"; one
+    group: no grouping); the weights are s of the chosen (without the correction), divided by their sum + 1e-20, times
+    `weight_scale`.  `identity`: that many further router outputs, behind the experts', belong to identity
     experts, which have no tensors and return their input; they take part in scores, groups and choice like the others.
     `routing="sigmoid"`: s = sigmoid(z); chosen are the `top` largest; the weights are the chosen scores as they are.
 
@@ -114,11 +115,11 @@ class MixtureOfExperts(Part):
                  router_bias: bool = True, names: Optional[dict] = None, gated: bool = True, activation: str = "silu",
                  routing: str = "top_logits", correction: bool = False, group_count: int = 1, group_keep: int = 1,
                  identity: int = 0, weight_scale: float = 1.0, weight_on: str = "output", limit: Optional[float] = None,
-                 act_alpha: float = 1.0):
+                 act_alpha: float = 1.0, score: str = "softmax", group_score: str = "max"):
         super().__init__(name, hidden_size=hidden_size, intermediate_size=intermediate_size, num_experts=num_experts, top=top,
                          router_bias=router_bias, gated=gated, activation=activation, routing=routing, correction=correction,
                          group_count=group_count, group_keep=group_keep, identity=identity, weight_scale=weight_scale,
-                         weight_on=weight_on, limit=limit, act_alpha=act_alpha)
+                         weight_on=weight_on, limit=limit, act_alpha=act_alpha, score=score, group_score=group_score)
         self.hidden, self.inter, self.E, self.top = int(hidden_size), int(intermediate_size), int(num_experts), int(top)
         self.identity = int(identity)
         self.outputs = self.E + self.identity                     # what the router puts out
@@ -144,6 +145,10 @@ class MixtureOfExperts(Part):
         self.has_correction = bool(correction)
         self.group_count, self.group_keep = max(1, int(group_count)), int(group_keep)
         self.weight_scale = float(weight_scale)
+        if score not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
+            raise ValueError(f"mixture of experts: scores are \"softmax\" or \"sigmoid\", a group's score \"max\" or \"top2\"; got "
+                             f"{score!r}, {group_score!r}")
+        self.score, self.group_score = score, group_score
         if routing != "scores" and (self.identity or self.has_correction or self.group_count > 1 or self.weight_scale != 1.0):
             raise ValueError("mixture of experts: identity experts, a correction, groups and a weight scale belong to routing=\"scores\"")
         if self.group_count > 1:
@@ -212,7 +217,7 @@ class MixtureOfExperts(Part):
         weights = rt.empty(n, self.top, dtype=torch.float32)
         if self.routing == "scores":
             kernels.moe_route_scored(h, self.router, self.correction, self.top, self.group_count, self.group_keep,
-                                     self.weight_scale, ids, weights)
+                                     self.weight_scale, ids, weights, score=self.score, group_score=self.group_score)
         else:
             # logits, choice and weights in one kernel
             kernels.moe_route(h, self.router_bias, self.top, ids, weights, router=self.router,

@@ -49,33 +49,40 @@ class RMSNorm(Part):
 
 @register_part("norm", "layernorm")
 class LayerNorm(Part):
-    """Layer norm with a gain and no bias: (v - mean) / sqrt(var + eps) · w, var the mean of the squared deviations,
-    statistics in float32.  Two uses: `forward`, the norm of the stream (as `RMSNorm.forward`: adds `delta` first),
-    and `add_normed`, for arrangements that normalise a branch's output before it joins the stream.  `tensor` is the
-    gain's name below the part's prefix."""
+    """Layer norm: (v - mean) / sqrt(var + eps) · w (+ b), var the mean of the squared deviations, statistics in float32.
+    Two uses: `forward`, the norm of the stream (as `RMSNorm.forward`: adds `delta` first, or the weighted sum of the
+    tokens' expert rows), and `add_normed`, for arrangements that normalise a branch's output before it joins the stream.
+    `tensor` is the gain's name below the part's prefix; `bias`: the suffix under which a bias is stored beside it (None:
+    the norm has no bias)."""
     graph_safe = True
+    takes_expert_rows = True
 
-    def __init__(self, name: str, size: int, eps: float, tensor: str = "weight"):
-        super().__init__(name, size=size, eps=eps, tensor=tensor)
+    def __init__(self, name: str, size: int, eps: float, tensor: str = "weight", bias: Optional[str] = None):
+        super().__init__(name, size=size, eps=eps, tensor=tensor, bias=bias)
         self.size = int(size)
         self.eps = float(eps)
         self.tensor = self.name + tensor
+        self.t_bias = self.tensor + bias if bias is not None else None
+        self.bias: Optional[torch.Tensor] = None
 
     def tensors(self):
-        return [TensorSpec(self.tensor, (self.size,), role="gain", init="one_plus_normal")]
+        specs = [TensorSpec(self.tensor, (self.size,), role="gain", init="one_plus_normal")]
+        return specs + ([TensorSpec(self.t_bias, (self.size,), role="bias")] if self.t_bias is not None else [])
 
     def bind(self, get, runtime):
         super().bind(get, runtime)
         self.gain = get(self.tensor).to(torch.float32).contiguous()
+        self.bias = get(self.t_bias).to(torch.float32).contiguous() if self.t_bias is not None else None
 
     def weight_bytes(self) -> int:
-        return self.gain.numel() * 4
+        return self.gain.numel() * (4 if self.bias is None else 8)
 
     def forward(self, x: torch.Tensor, delta: Optional[torch.Tensor] = None,
-                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-        """x: float32 [n, size], updated in place to x + delta when delta is given; returns LN(x)."""
+                out_dtype: Optional[torch.dtype] = None, expert_rows=None) -> torch.Tensor:
+        """x: float32 [n, size], updated in place to x + delta when delta is given, or to x plus the weighted sum of
+        `expert_rows` (see `kernels.layernorm`); returns LN(x)."""
         out = self.runtime.empty(*x.shape, dtype=out_dtype or self.runtime.dtype)
-        kernels.layernorm(x, delta, self.gain, self.eps, out, of_branch=False)
+        kernels.layernorm(x, delta, self.gain, self.eps, out, of_branch=False, bias=self.bias, expert_rows=expert_rows)
         return out
 
     def add_normed(self, x: torch.Tensor, y: torch.Tensor, copy_dtype: Optional[torch.dtype] = None
@@ -83,7 +90,7 @@ class LayerNorm(Part):
         """x (float32 [n, size], in place) += LN(y), y float32 [n, size] or slices [s, n, size] that are added up first.
         With `copy_dtype`, also returns the new x in that type (the next part's input)."""
         out = self.runtime.empty(*x.shape, dtype=copy_dtype) if copy_dtype is not None else None
-        kernels.layernorm(x, y, self.gain, self.eps, out, of_branch=True)
+        kernels.layernorm(x, y, self.gain, self.eps, out, of_branch=True, bias=self.bias)
         return out
 
 
