@@ -470,28 +470,42 @@ __global__ void layernorm_kernel(float* __restrict__ x, NormBranch br, const flo
 }
 
 // Many rows: a warp per row, the row in registers from the first load to the last store (NV 16-byte pieces per lane,
-// d <= 128 * NV, d a multiple of 4, all pointers 16-byte aligned); no shared memory and no block-wide barrier.
-template <typename T, int NV>
+// d <= 128 * NV, d a multiple of 4, all pointers 16-byte aligned).  The block's rows share gain and bias through shared
+// memory, copied there asynchronously ahead of everything else (left to the last loop, their loads would wait one by one
+// behind the row's registers).
+// BRANCH: 0 none, 1 slices, 2 expert rows; MODE: ln_mode.  (Forms of their own: only what a form needs takes registers.)
+template <typename T, int NV, int BRANCH, int MODE>
 __global__ void __launch_bounds__(256)
 layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restrict__ gain, const float* __restrict__ bias,
-                      float eps, int d, int n, int ln_mode, T* __restrict__ out) {
+                      float eps, int d, int n, T* __restrict__ out) {
+    extern __shared__ __align__(16) float affine[];        // [d] gain, then [d] bias (if there is one)
     grid_launch_dependents();
+    const int d4 = d >> 2;
+    for (int i = threadIdx.x; i < (bias != nullptr ? 2 : 1) * d4; i += blockDim.x) {
+        const float* src = i < d4 ? gain + 4 * i : bias + 4 * (i - d4);
+        const unsigned dst = (unsigned)__cvta_generic_to_shared(affine + 4 * i);
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src));
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
     grid_dependency_wait();
     const int lane = threadIdx.x & 31;
-    const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (row >= n) return;
+    const int row = min(blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), n - 1);
+    const bool live = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5) < n;       // the last block's spare warps only keep company
     const long long base = (long long)row * d;
-    const int d4 = d >> 2;
-    const bool has_branch = br.y != nullptr || br.rows != nullptr;
     float4* x4 = reinterpret_cast<float4*>(x + base);
-    float4 v[NV], xv[NV];
+    float4 v[NV], xv[MODE == 1 ? NV : 1];              // MODE 1 keeps the stream's entries beside the branch's
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = lane + 32 * k;
-        xv[k] = (i < d4) ? x4[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        v[k] = (ln_mode == 0) ? xv[k] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float4 xi = live && i < d4 ? x4[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if constexpr (MODE == 0) {
+            v[k] = xi;
+        } else {
+            xv[k] = xi;
+            v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
     }
-    if (br.y != nullptr) {
+    if constexpr (BRANCH == 1) {
         for (int s = 0; s < br.n_slices; ++s) {
             const float4* t4 = reinterpret_cast<const float4*>(br.y + s * br.slice_stride + base);
 #pragma unroll
@@ -504,10 +518,7 @@ layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restr
             }
         }
     }
-    if (br.rows != nullptr) {
-        float4 acc[NV];
-#pragma unroll
-        for (int k = 0; k < NV; ++k) acc[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if constexpr (BRANCH == 2) {
         for (int j = 0; j < br.top; ++j) {
             const float w = br.weights[(long long)row * br.top + j];
             const float4* t4 = reinterpret_cast<const float4*>(br.rows + (long long)br.row_of[(long long)row * br.top + j] * d);
@@ -516,13 +527,11 @@ layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restr
                 const int i = lane + 32 * k;
                 if (i < d4) {
                     const float4 t = __ldg(t4 + i);
-                    acc[k].x = fmaf(w, t.x, acc[k].x); acc[k].y = fmaf(w, t.y, acc[k].y);
-                    acc[k].z = fmaf(w, t.z, acc[k].z); acc[k].w = fmaf(w, t.w, acc[k].w);
+                    v[k].x = fmaf(w, t.x, v[k].x); v[k].y = fmaf(w, t.y, v[k].y);
+                    v[k].z = fmaf(w, t.z, v[k].z); v[k].w = fmaf(w, t.w, v[k].w);
                 }
             }
         }
-#pragma unroll
-        for (int k = 0; k < NV; ++k) { v[k].x += acc[k].x; v[k].y += acc[k].y; v[k].z += acc[k].z; v[k].w += acc[k].w; }
     }
     float sum = 0.0f;
 #pragma unroll
@@ -537,21 +546,24 @@ layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restr
         }
     }
     const float rstd = 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
-    const float4* g4 = reinterpret_cast<const float4*>(gain);
-    const float4* b4 = reinterpret_cast<const float4*>(bias);
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();
+    if (!live) return;
+    const float4* g4 = reinterpret_cast<const float4*>(affine);
+    const float4* b4 = bias != nullptr ? g4 + d4 : nullptr;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = lane + 32 * k;
         if (i >= d4) continue;
-        const float4 g = __ldg(g4 + i);
+        const float4 g = g4[i];
         float r[4] = {(v[k].x - mean) * rstd * g.x, (v[k].y - mean) * rstd * g.y, (v[k].z - mean) * rstd * g.z,
                       (v[k].w - mean) * rstd * g.w};
         if (b4 != nullptr) {
-            const float4 b = __ldg(b4 + i);
+            const float4 b = b4[i];
             r[0] += b.x; r[1] += b.y; r[2] += b.z; r[3] += b.w;
         }
-        if (ln_mode == 0) {
-            if (has_branch) x4[i] = v[k];
+        if constexpr (MODE == 0) {
+            if constexpr (BRANCH != 0) x4[i] = v[k];
         } else {
             r[0] += xv[k].x; r[1] += xv[k].y; r[2] += xv[k].z; r[3] += xv[k].w;
             x4[i] = make_float4(r[0], r[1], r[2], r[3]);
@@ -561,14 +573,25 @@ layernorm_warp_kernel(float* __restrict__ x, NormBranch br, const float* __restr
     }
 }
 
+template <typename T, int BRANCH, int MODE>
+static cudaError_t launch_layernorm_warp(int nv, float* x, const NormBranch& br, const float* gain, const float* bias, float eps,
+                                         int d, int n, T* out, cudaStream_t s) {
+    auto k = nv <= 1 ? layernorm_warp_kernel<T, 1, BRANCH, MODE> : nv <= 2 ? layernorm_warp_kernel<T, 2, BRANCH, MODE>
+           : nv <= 4 ? layernorm_warp_kernel<T, 4, BRANCH, MODE> : nv <= 8 ? layernorm_warp_kernel<T, 8, BRANCH, MODE>
+           : layernorm_warp_kernel<T, 12, BRANCH, MODE>;
+    return launch_pdl(k, dim3((n + 7) / 8), dim3(256), (size_t)d * sizeof(float) * (bias != nullptr ? 2 : 1), s, x, br,
+                      gain, bias, eps, d, n, out);
+}
+
 template <typename T>
 static cudaError_t launch_layernorm(bool vec, int nv, float* x, const NormBranch& br, const float* gain, const float* bias, float eps,
                                     int d, int n, int ln_mode, T* out, size_t smem, int threads, cudaStream_t s) {
     if (vec && nv <= 12 && n >= 128) {
-        const dim3 grid((n + 7) / 8), block(256);
-        auto k = nv <= 1 ? layernorm_warp_kernel<T, 1> : nv <= 2 ? layernorm_warp_kernel<T, 2> : nv <= 4 ? layernorm_warp_kernel<T, 4>
-               : nv <= 8 ? layernorm_warp_kernel<T, 8> : layernorm_warp_kernel<T, 12>;
-        return launch_pdl(k, grid, block, 0, s, x, br, gain, bias, eps, d, n, ln_mode, out);
+        if (ln_mode == 0 && br.rows != nullptr) return launch_layernorm_warp<T, 2, 0>(nv, x, br, gain, bias, eps, d, n, out, s);
+        if (ln_mode == 0 && br.y != nullptr) return launch_layernorm_warp<T, 1, 0>(nv, x, br, gain, bias, eps, d, n, out, s);
+        if (ln_mode == 0) return launch_layernorm_warp<T, 0, 0>(nv, x, br, gain, bias, eps, d, n, out, s);
+        if (br.rows != nullptr) return launch_layernorm_warp<T, 2, 1>(nv, x, br, gain, bias, eps, d, n, out, s);
+        return launch_layernorm_warp<T, 1, 1>(nv, x, br, gain, bias, eps, d, n, out, s);
     }
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {

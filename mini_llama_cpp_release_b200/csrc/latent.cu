@@ -8,7 +8,9 @@
 // which is attention with one key/value head of size rank + rot that every query head reads, values being the first
 // `rank` entries of the key rows.  Two kernels here: `latent_prepare` (norm of the latent, rotation of the shared key
 // part and of the queries' rotated parts, the cache write) and `head_project` (a small matrix product per head, for
-// the two moved expansions), both with float32 arithmetic.
+// the two moved expansions), both with float32 arithmetic.  `head_project` has a second form for 16-bit weights on the
+// tensor cores (mma.sync: the operands are a few megabytes at most, so what counts is that every load of a tile is in flight
+// at once); its float32 inputs enter as the sum of two 16-bit numbers.
 #include "common.cuh"
 
 namespace mlc {
@@ -138,6 +140,161 @@ head_project_kernel(const TI* __restrict__ in, long long in_st, long long in_sh,
     }
 }
 
+// ---- the same product on the tensor cores: W in bfloat16, accumulation in float32.
+__device__ __forceinline__ void hp_ldmatrix(unsigned (&r)[4], const bf16* p) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
+}
+__device__ __forceinline__ void hp_ldmatrix_trans(unsigned (&r)[4], const bf16* p) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
+}
+__device__ __forceinline__ void hp_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+struct HeadProjectArgs {
+    const void* in;
+    long long in_st, in_sh;
+    const bf16* w;
+    long long w_sh;
+    long long w_ld;             // elements between W's rows: [j][d] rows of d, or [d][j] rows of j
+    bf16* out;
+    long long out_st, out_sh;
+    int n, n_in, n_out;
+    const float* gate;
+    long long gate_st;
+};
+
+// A block: TM tokens x 64 outputs of one head, four warps.  TM = 64: warp w takes tokens 16w .. 16w+15 and all 64 outputs;
+// TM = 16: all warps take the 16 tokens, warp w outputs 16w .. 16w+15.  The inner size is walked in chunks of KC, each staged
+// in shared memory by 16-byte loads (sizes, strides and addresses allow them: the host sees to it).  A float32 input x is
+// staged as hi + lo, hi = x rounded to bfloat16 and lo = x - hi rounded, and both meet the weights.  An output's products are
+// added in the same order whatever TM.  BY_D: W's rows hold d contiguously ([j][d]); else [d][j].
+template <typename TI, int TM, bool BY_D>
+__global__ void __launch_bounds__(128)
+head_project_mma_kernel(HeadProjectArgs a) {
+    constexpr int KC = TM == 16 ? 128 : 64;
+    constexpr int XS = KC + 8, WS = BY_D ? KC + 8 : 64 + 8;
+    constexpr bool SPLIT = sizeof(TI) == 4;
+    constexpr int NT = TM == 16 ? 1 : 4;                   // pairs of 8-output tiles a warp owns
+    __shared__ __align__(16) bf16 xs[(SPLIT ? 2 : 1) * TM * XS];
+    __shared__ __align__(16) bf16 ws[BY_D ? 64 * WS : KC * WS];
+    const int h = blockIdx.z, t0 = blockIdx.y * TM, j0 = blockIdx.x * 64;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int row0 = TM == 16 ? 0 : 16 * warp, col0 = TM == 16 ? 16 * warp : 0;
+    const TI* in = (const TI*)a.in + (long long)h * a.in_sh;
+    const bf16* w = a.w + (long long)h * a.w_sh;
+    float acc[2 * NT][4];
+#pragma unroll
+    for (int i = 0; i < 2 * NT; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) acc[i][k] = 0.0f;
+    grid_launch_dependents();
+    for (int d0 = 0; d0 < a.n_in; d0 += KC) {
+        if (d0 > 0) __syncthreads();
+        // the weights' chunk: they depend on no kernel before this one
+        constexpr int W_ROWS = BY_D ? 64 : KC, W_PACKS = (BY_D ? KC : 64) / 8;
+#pragma unroll
+        for (int idx = tid; idx < W_ROWS * W_PACKS; idx += 128) {
+            const int r = idx / W_PACKS, c = (idx % W_PACKS) * 8;
+            const int j = j0 + (BY_D ? r : c), d = d0 + (BY_D ? c : r);
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (j < a.n_out && d < a.n_in) v = *reinterpret_cast<const uint4*>(w + (BY_D ? j * a.w_ld + d : d * a.w_ld + j));
+            *reinterpret_cast<uint4*>(ws + r * WS + c) = v;
+        }
+        if (d0 == 0) grid_dependency_wait();
+#pragma unroll
+        for (int idx = tid; idx < TM * (KC / 8); idx += 128) {
+            const int r = idx / (KC / 8), c = (idx % (KC / 8)) * 8;
+            const bool ok = t0 + r < a.n && d0 + c < a.n_in;
+            const TI* p = in + (long long)(t0 + r) * a.in_st + d0 + c;
+            if constexpr (SPLIT) {
+                float4 u = make_float4(0.0f, 0.0f, 0.0f, 0.0f), v = u;
+                if (ok) {
+                    u = *reinterpret_cast<const float4*>(p);
+                    v = *reinterpret_cast<const float4*>(p + 4);
+                }
+                const float f[8] = {u.x, u.y, u.z, u.w, v.x, v.y, v.z, v.w};
+                __align__(16) bf16 hi[8], lo[8];
+#pragma unroll
+                for (int k = 0; k < 8; ++k) {
+                    hi[k] = __float2bfloat16_rn(f[k]);
+                    lo[k] = __float2bfloat16_rn(f[k] - __bfloat162float(hi[k]));
+                }
+                *reinterpret_cast<uint4*>(xs + r * XS + c) = *reinterpret_cast<const uint4*>(hi);
+                *reinterpret_cast<uint4*>(xs + (TM + r) * XS + c) = *reinterpret_cast<const uint4*>(lo);
+            } else {
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (ok) v = *reinterpret_cast<const uint4*>(p);
+                *reinterpret_cast<uint4*>(xs + r * XS + c) = v;
+            }
+        }
+        __syncthreads();
+        const int k_end = min(KC, (a.n_in - d0 + 15) & ~15);       // what lies beyond n_in is zero
+        for (int k = 0; k < k_end; k += 16) {
+            unsigned ah[4], al[4];
+            hp_ldmatrix(ah, xs + (row0 + (lane & 15)) * XS + k + (lane >> 4) * 8);
+            if constexpr (SPLIT) hp_ldmatrix(al, xs + (TM + row0 + (lane & 15)) * XS + k + (lane >> 4) * 8);
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                unsigned b[4];
+                const int c = col0 + 16 * t;
+                if constexpr (BY_D) hp_ldmatrix(b, ws + (c + (lane >> 4) * 8 + (lane & 7)) * WS + k + ((lane >> 3) & 1) * 8);
+                else hp_ldmatrix_trans(b, ws + (k + (lane & 15)) * WS + c + (lane >> 4) * 8);
+                hp_mma(acc[2 * t], ah, b[0], b[1]);
+                hp_mma(acc[2 * t + 1], ah, b[2], b[3]);
+                if constexpr (SPLIT) {
+                    hp_mma(acc[2 * t], al, b[0], b[1]);
+                    hp_mma(acc[2 * t + 1], al, b[2], b[3]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * NT; ++i) {
+        const int j = j0 + col0 + 8 * i + (lane & 3) * 2;
+        if (j >= a.n_out) continue;                        // n_out is even
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int t = t0 + row0 + (lane >> 2) + 8 * half;
+            if (t >= a.n) continue;
+            float u = acc[i][2 * half], v = acc[i][2 * half + 1];
+            if (a.gate != nullptr) {
+                const float* g = a.gate + t * a.gate_st + (long long)h * a.n_out + j;
+                u /= 1.0f + expf(-g[0]);
+                v /= 1.0f + expf(-g[1]);
+            }
+            *reinterpret_cast<__nv_bfloat162*>(a.out + t * a.out_st + h * a.out_sh + j) = __floats2bfloat162_rn(u, v);
+        }
+    }
+}
+
+// Whether the tensor-core form takes these operands: 16-byte loads along each operand's contiguous direction, paired stores.
+static bool head_project_mma_takes(const void* in, int in_dtype, long long in_st, long long in_sh, const void* w, long long w_sh,
+                                   long long w_sd, long long w_sj, const void* out, long long out_st, long long out_sh, int n_in,
+                                   int n_out) {
+    const int in_pack = in_dtype == MLC_DTYPE_F32 ? 4 : 8;
+    const bool by_d = w_sd == 1;
+    if (!by_d && w_sj != 1) return false;
+    const long long w_ld = by_d ? w_sj : w_sd;
+    if (n_in % 8 != 0 || (by_d ? n_out % 2 : n_out % 8) != 0) return false;
+    if (w_ld % 8 != 0 || w_sh % 8 != 0 || in_st % in_pack != 0 || in_sh % in_pack != 0 || out_st % 2 != 0 || out_sh % 2 != 0) return false;
+    return ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(w)) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 3) == 0;
+}
+
+template <typename TI>
+static cudaError_t launch_head_project_mma(const HeadProjectArgs& a, bool by_d, int H, cudaStream_t s) {
+    const int tm = a.n <= 16 ? 16 : 64;
+    const dim3 grid((a.n_out + 63) / 64, (a.n + tm - 1) / tm, H), block(128);
+    if (tm == 16) return launch_pdl(by_d ? head_project_mma_kernel<TI, 16, true> : head_project_mma_kernel<TI, 16, false>, grid, block, 0, s, a);
+    return launch_pdl(by_d ? head_project_mma_kernel<TI, 64, true> : head_project_mma_kernel<TI, 64, false>, grid, block, 0, s, a);
+}
+
 }  // namespace mlc
 
 using namespace mlc;
@@ -176,6 +333,15 @@ extern "C" int mlc_head_project(const void* in, int in_dtype, long long in_st, l
     const dim3 grid((n_out + HP_TILE - 1) / HP_TILE, (n + HP_TILE - 1) / HP_TILE, H);
     if (grid.y > 65535) return MLC_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
+    if (w_dtype == MLC_DTYPE_BF16 && out_dtype == MLC_DTYPE_BF16 &&
+        head_project_mma_takes(in, in_dtype, in_st, in_sh, w, w_sh, w_sd, w_sj, out, out_st, out_sh, n_in, n_out)) {
+        const bool by_d = w_sd == 1;
+        const HeadProjectArgs a{in, in_st, in_sh, (const bf16*)w, w_sh, by_d ? w_sj : w_sd, (bf16*)out, out_st, out_sh, n, n_in,
+                                n_out, gate, gate_st};
+        const cudaError_t e = in_dtype == MLC_DTYPE_F32 ? launch_head_project_mma<float>(a, by_d, H, s)
+                                                        : launch_head_project_mma<bf16>(a, by_d, H, s);
+        return e == cudaSuccess ? 0 : (int)e;
+    }
     const int code = in_dtype * 4 + w_dtype * 2 + out_dtype;
 #define MLC_HP(TI, TW, TO)                                                                                                  \
     head_project_kernel<TI, TW, TO><<<grid, 256, 0, s>>>((const TI*)in, in_st, in_sh, (const TW*)w, w_sh, w_sd, w_sj, (TO*)out, \

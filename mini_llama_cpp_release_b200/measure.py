@@ -112,6 +112,36 @@ def _nobonex(width: int, ff: int, heads: int, kv_heads: int, head: int, n_layers
             "embedding": {"scale": 4.0}, "layers": layers}
 
 
+def _bizenex(width: int, ff: int, heads: int, kv_heads: int, head: int, n_layers: int, vocab: int, design: str = "Bizenex") -> Dict[str, Any]:
+    """Bizenex layers of real width in a cycle of six: attention, latent attention, latent attention on the latents of the
+    layer before it, attention twice, latent attention; every layer has experts.  The attention's shape (heads, kv heads,
+    head size) and the width are the Qwen2 preset's of the same width, the experts (eight of half its dense feed-forward, two
+    chosen; here in four groups of which two are kept) and the cached latent row of 128 entries are the Kebesun preset's.
+    `design="Kebesun"` gives that design's layers of the same mixers and sizes in the same order (attention without norms,
+    sinks and temperature, rotated; latent attention of 80 plain and 48 rotated entries without sink, gate and sharing;
+    experts without groups): the model the Bizenex preset is timed beside."""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5}
+    lat = {"heads": heads, "dim": head, "vdim": head, "kv_rank": 128, "scale": head ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+    if design == "Kebesun":
+        rot = {"dims": head, "base": 1000000.0, "scaling": {"factor": 4.0}}
+        att = dict(att, rot=rot)
+        lat = dict(lat, kv_rank=80, rot_dim=48, scale=(head + 48) ** -0.5, rot=dict(rot, dims=48))
+        top = {"architecture": "Kebesun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}}
+    else:
+        att = dict(att, q_temp={"coef": 0.1, "every": 1024})
+        moe["router"] = dict(moe["router"], groups={"count": 4, "keep": 2})
+        top = {"architecture": "Bizenex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0}
+    layers = []
+    for i in range(n_layers):
+        t = ("attention", "latent_attention", "latent_attention", "attention", "attention", "latent_attention")[i % 6]
+        m = dict(att if t == "attention" else lat)
+        if i % 6 == 2 and design == "Bizenex":
+            m["kv_from"] = i - 1
+        layers.append({"type": t, "mixer": m, "mlp": dict(moe)})
+    return dict(top, layers=layers)
+
+
 PRESETS: Dict[str, Dict[str, Any]] = {
     "tiny-a": dict(_QWEN2, hidden_size=64, intermediate_size=176, num_hidden_layers=2, num_attention_heads=4,
                    num_key_value_heads=2, head_dim=16, vocab_size=512, max_position_embeddings=256, rope_theta=10000.0,
@@ -147,6 +177,13 @@ PRESETS: Dict[str, Dict[str, Any]] = {
     "nobonex-w896": _nobonex(896, 4864, 14, 2, 64, 24, 151936),
     "nobonex-w1536": _nobonex(1536, 8960, 12, 2, 128, 24, 151936),
     "nobonex-w3584": _nobonex(3584, 18944, 28, 4, 128, 24, 152064),
+    # the Bizenex design at the same widths, and the Kebesun layers of the same mixers it is timed beside (see `_bizenex`)
+    "bizenex-w896": _bizenex(896, 4864, 14, 2, 64, 24, 151936),
+    "bizenex-w1536": _bizenex(1536, 8960, 12, 2, 128, 24, 151936),
+    "bizenex-w3584": _bizenex(3584, 18944, 28, 4, 128, 24, 152064),
+    "kebesun-al-w896": _bizenex(896, 4864, 14, 2, 64, 24, 151936, design="Kebesun"),
+    "kebesun-al-w1536": _bizenex(1536, 8960, 12, 2, 128, 24, 151936, design="Kebesun"),
+    "kebesun-al-w3584": _bizenex(3584, 18944, 28, 4, 128, 24, 152064, design="Kebesun"),
 }
 
 FALLBACK_PEAKS = dict(hbm_gbs=6650.0, bf16_tflops=1590.0)
