@@ -65,12 +65,13 @@ def plan_groups(needs: Sequence[Optional[CacheNeed]], reads_cache_of: Sequence[O
                     needs[e].kv_heads != needs[src].kv_heads or needs[e].head_dim != needs[src].head_dim):
                 raise ValueError(f"schedule entry {e} cannot read the cache of entry {src}: kv heads or head size differ")
             if needs[e] is not None and needs[src] is not None and needs[src].kind == "window" and (
-                    needs[e].kind != "window" or (needs[e].window or 0) > (needs[src].window or 0)):
+                    needs[e].kind != "window" or (needs[e].window or 0) > (needs[src].window or 0)
+                    or needs[e].keep_first > needs[src].keep_first):
                 # the owner gives pages back once its own window has passed them; a reader that looks further back
                 # would find them gone
                 raise ValueError(f"schedule entry {e} cannot read the cache of entry {src}: it reads "
-                                 f"{'all keys' if needs[e].kind != 'window' else f'a window of {needs[e].window}'}, "
-                                 f"the owner keeps a window of {needs[src].window}")
+                                 f"{'all keys' if needs[e].kind != 'window' else f'a window of {needs[e].window} and the first {needs[e].keep_first}'}, "
+                                 f"the owner keeps a window of {needs[src].window} and the first {needs[src].keep_first}")
             if needs[e] is not None and needs[src] is not None and needs[src].kind == "chunk" and (
                     needs[e].kind != "chunk" or needs[e].window != needs[src].window):
                 # the owner gives a chunk's pages back once the sequence has left the chunk

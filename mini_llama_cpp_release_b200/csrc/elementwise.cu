@@ -8,6 +8,7 @@
 // (i, i + hd/2) (src/ops.cpp:125-141), gate·(1/(1+exp(-gate)))·up (src/ops.cpp:94-107),
 // the residual sum (src/forward.cpp:772, 779).  What is new is the fusion and the layout.
 #include "common.cuh"
+#include "norm_branch.cuh"
 
 namespace mlc {
 
@@ -327,71 +328,7 @@ __global__ void convert_kernel(const TIn* __restrict__ in, long long total, TOut
 // ln_mode 0, "norm of the stream":   x += branch (if any);  out = LN(x)            (out in T)
 // ln_mode 1, "norm of the branch":   x += LN(branch);       out = x, if asked for  (out in T)
 //
-// The branch is y, float32 slices added in order, or the weighted sum of a token's expert rows,
-// sum_j weights[t][j] · rows[row_of[t][j]], j in the order of the choices.
-struct NormBranch {
-    const float* y;             // [n_slices][n][d], or null
-    int n_slices;
-    long long slice_stride;
-    const float* rows;          // expert rows [.][d], or null
-    const int* row_of;          // [n][top]
-    const float* weights;       // [n][top]
-    int top;
-};
-
-struct Four { float e[4]; };
-__device__ __forceinline__ Four load_four(const float* p) {
-    const float4 t = *reinterpret_cast<const float4*>(p);
-    return Four{{t.x, t.y, t.z, t.w}};
-}
-
-// v (VEC entries of row t from entry i on) += the branch's entries
-template <int VEC>
-__device__ __forceinline__ void add_branch(const NormBranch& br, long long t, int d, int i, float (&v)[VEC]) {
-    if (br.y != nullptr) {
-        const float* p = br.y + t * d + i;
-#pragma unroll 8
-        for (int s = 0; s < br.n_slices; ++s) {
-            if constexpr (VEC == 4) {
-                const Four q = load_four(p + s * br.slice_stride);
-#pragma unroll
-                for (int k = 0; k < VEC; ++k) v[k] += q.e[k];
-            } else {
-                v[0] += __ldg(p + s * br.slice_stride);
-            }
-        }
-    }
-    if (br.rows != nullptr) {
-        float acc[VEC];
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) acc[k] = 0.0f;
-#pragma unroll 4
-        for (int j = 0; j < br.top; ++j) {
-            const float w = br.weights[t * br.top + j];
-            const float* p = br.rows + (long long)br.row_of[t * br.top + j] * d + i;
-            if constexpr (VEC == 4) {
-                const Four q = load_four(p);
-#pragma unroll
-                for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w, q.e[k], acc[k]);
-            } else {
-                acc[0] = fmaf(w, *p, acc[0]);
-            }
-        }
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) v[k] += acc[k];
-    }
-}
-
-template <typename T>
-__device__ __forceinline__ void store_four(T* p, const float (&r)[4]) {
-    if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]);
-    } else {
-        __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
-        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
-    }
-}
-
+// The branch: see norm_branch.cuh.
 // A block per row; the row waits in shared memory between the passes.  VEC 4: 16-byte accesses (rows whose length is a
 // multiple of 4, all pointers 16-byte aligned); VEC 1: any row, and few rows, where one entry a thread has more loads in flight.
 template <typename T, int VEC>
@@ -618,7 +555,9 @@ static cudaError_t launch_layernorm(bool vec, int nv, float* x, const NormBranch
 // none); `whole_row`: the norm's statistic is taken over all query heads together (and over all key heads together) and the
 // gains are as long as the projection, instead of one statistic per head and a gain shared by the heads; `interleaved`: the
 // rotation pairs entry 2j with 2j + 1 instead of entry j with j + dims/2; `temp_every` > 0: the queries of position p are
-// multiplied by 1 + temp_coef · ln(floor((p + 1) / temp_every) + 1).
+// multiplied by 1 + temp_coef · ln(floor((p + 1) / temp_every) + 1).  `maps` > 1 (differential attention): a key head holds
+// that many keys of `dim` entries side by side, each normed and rotated by itself, and query head h meets only the (h % maps)-th
+// of them: its entries lie at that place of its row, zeros elsewhere.
 struct QkOptions {
     const float* q_bias;
     const float* k_bias;
@@ -627,6 +566,7 @@ struct QkOptions {
     int interleaved;
     float temp_coef;
     int temp_every;
+    int maps;
 };
 
 template <typename T>
@@ -643,7 +583,8 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
     const int seq = tok_seq[n];
     const int half = rot_dims >> 1;
     const float2* cs = (rope != nullptr && half > 0) ? rope + (long long)min(p, rope_positions - 1) * half : nullptr;
-    const int n_heads = q_heads + 2 * kv_heads_in_row;
+    const int maps = opt.maps, k_units = maps * kv_heads_in_row;         // a unit: `dim` projected entries with a norm of their own
+    const int n_heads = q_heads + k_units + kv_heads_in_row;
     const float q_temp = opt.temp_every > 0 ? 1.0f + opt.temp_coef * logf((float)((p + 1) / opt.temp_every) + 1.0f) : 1.0f;
     // a norm over the whole projection: one statistic for all query heads and one for all key heads, summed in an order
     // that the row's length alone fixes (a thread a strided share, then the block's tree)
@@ -658,15 +599,15 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
         f_q = 1.0f / sqrtf(block_sum(ss, scratch) / (float)(q_heads * dim) + eps);
         if (kv_heads_in_row > 0) {
             ss = 0.0f;
-            for (int i = threadIdx.x; i < kv_heads_in_row * dim; i += blockDim.x) {
+            for (int i = threadIdx.x; i < k_units * dim; i += blockDim.x) {
                 const float v = row[k_col + i] + (opt.k_bias != nullptr ? opt.k_bias[i] : 0.0f);
                 ss += v * v;
             }
-            f_k = 1.0f / sqrtf(block_sum(ss, scratch) / (float)(kv_heads_in_row * dim) + eps);
+            f_k = 1.0f / sqrtf(block_sum(ss, scratch) / (float)(k_units * dim) + eps);
         }
     }
     for (int head = warp; head < n_heads; head += n_warps) {
-        if (head < q_heads + kv_heads_in_row) {
+        if (head < q_heads + k_units) {
             const bool is_q = head < q_heads;
             const int h = is_q ? head : head - q_heads;
             const float* src = row + (is_q ? q_col : k_col) + h * dim;
@@ -675,7 +616,10 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
             const float* gain = is_q ? q_gain : k_gain;
             if (gain != nullptr && opt.whole_row) gain += h * dim;             // a gain as long as the projection
             T* dst = is_q ? q_out + ((long long)n * q_heads + head) * D
-                          : (T*)cache.k_pool + paged_offset(cache, seq, p, h);
+                          : (T*)cache.k_pool + paged_offset(cache, seq, p, h / maps);
+            // the unit's place in its row, and the part of the row this unit writes (zeros where it has no entries)
+            const int place = (h % maps) * dim;
+            const int from = is_q ? 0 : place, to = is_q || h % maps == maps - 1 ? D : place + dim;
             float f = is_q ? f_q : f_k;
             if (!opt.whole_row) {
                 float ss = 0.0f;
@@ -687,9 +631,10 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
                 f = eps >= 0.0f ? 1.0f / sqrtf(ss / (float)dim + eps) : 1.0f;      // a negative eps: no norm
             }
             if (is_q) f *= q_temp;              // the rotation is linear: the factor acts on both entries of a pair
-            for (int i = lane; i < D; i += 32) {
+            for (int at = from + lane; at < to; at += 32) {
+                const int i = at - place;
                 float v = 0.0f;
-                if (i < dim) {
+                if (i >= 0 && i < dim) {
                     const float raw = src[i] + (bias != nullptr ? bias[i] : 0.0f);
                     v = gain != nullptr ? raw * f * gain[i] : raw * f;
                     if (cs != nullptr && i < rot_dims) {
@@ -704,10 +649,10 @@ __global__ void qk_norm_rope_cache_kernel(const float* __restrict__ proj, long l
                         v = first ? v * t.x - w * t.y : v * t.x + w * t.y;
                     }
                 }
-                dst[i] = from_float<T>(v);
+                dst[at] = from_float<T>(v);
             }
         } else {
-            const int vh = head - q_heads - kv_heads_in_row;
+            const int vh = head - q_heads - k_units;
             const float* src = row + v_col + vh * vdim;
             const float* bias = opt.v_bias != nullptr ? opt.v_bias + vh * vdim : nullptr;
             T* dst = (T*)cache.v_pool + paged_offset(cache, seq, p, vh);
@@ -819,15 +764,15 @@ extern "C" int mlc_qk_norm_rope_cache(const float* proj, long long stride, int q
                                       void* k_pool, void* v_pool, const int* page_table, long long entry_offset,
                                       int pages_per_seq, int page_size, int cache_kv_heads, const float* q_bias,
                                       const float* k_bias, const float* v_bias, int whole_row, int interleaved, float temp_coef,
-                                      int temp_every, void* stream) {
+                                      int temp_every, int maps, void* stream) {
     if (n <= 0) return 0;
-    const QkOptions opt{q_bias, k_bias, v_bias, whole_row, interleaved, temp_coef, temp_every};
-    if (dim <= 0 || vdim <= 0 || D < dim || D < vdim || q_heads <= 0 || kv_heads_in_row < 0) return MLC_ERR_BAD_SIZE;
+    const QkOptions opt{q_bias, k_bias, v_bias, whole_row, interleaved, temp_coef, temp_every, maps};
+    if (maps < 1 || dim <= 0 || vdim <= 0 || D < maps * dim || D < vdim || q_heads <= 0 || q_heads % maps || kv_heads_in_row < 0) return MLC_ERR_BAD_SIZE;
     if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim) return MLC_ERR_BAD_SIZE;
     if (kv_heads_in_row != 0 && kv_heads_in_row != cache_kv_heads) return MLC_ERR_BAD_SIZE;
     PagedKV c{k_pool, v_pool, page_table, entry_offset, pages_per_seq, page_size, cache_kv_heads, D};
     cudaStream_t s = (cudaStream_t)stream;
-    const int heads = q_heads + 2 * kv_heads_in_row;
+    const int heads = q_heads + (maps + 1) * kv_heads_in_row;
     const int threads = 32 * (heads < 8 ? heads : 8);
     if (dtype == MLC_DTYPE_F32)
         qk_norm_rope_cache_kernel<float><<<n, threads, 0, s>>>(proj, stride, q_col, k_col, v_col, q_gain, k_gain, eps, positions,

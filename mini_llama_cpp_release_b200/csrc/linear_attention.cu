@@ -18,6 +18,7 @@
 // sequence still spreads over the GPU.  Tokens that are not there count as q = k = v = 0 with a
 // decay of one.  State layout in a slot's row: [head][column][row] (a column's rows side by side).
 #include "common.cuh"
+#include "linear_attention.cuh"
 
 namespace mlc {
 
@@ -25,30 +26,6 @@ constexpr int GLA_CHUNK = 16;      // tokens staged at a time
 constexpr int GLA_COLS = 16;       // columns of S per block
 constexpr int GLA_THREADS = 64;    // 8 pairs of columns x 8 groups of rows
 constexpr int GLA_V_LOADS = GLA_CHUNK * GLA_COLS / GLA_THREADS;
-
-struct GlaArgs {
-    const float* qk;            // rows that hold q (at q_col) and k (at k_col)
-    long long qk_stride;
-    const float* vsrc;          // rows that hold v (at v_col); may be the same matrix
-    long long v_stride;
-    int q_col, k_col, v_col;
-    const float* decay;         // [n][H*dim] decays
-    float q_scale;
-    float* state;               // [slots][H*vdim*dim]
-    long long state_stride;
-    const int* slots;
-    const int* cu_seqlens;
-    float* out;                 // [row slabs][n][H*vdim]
-    long long out_slice;        // floats between the slices of two row slabs
-    int H, dim, vdim;
-    int col_slabs;
-    // a state-space layer's use of the walk: `qk_share` heads in a row read the same q and k (head h reads group h / qk_share;
-    // 1: every head its own), `head_decay` [n][H] is one decay per token and head for all of a head's rows (then `decay` is
-    // not read), `v_scale` [n][H] multiplies the head's v as it is read.  Null: the ordinary forms.
-    int qk_share;
-    const float* head_decay;
-    const float* v_scale;
-};
 
 // z <- sigmoid(z + bias)^(1/tau) = exp(logsigmoid(z + bias) / tau),  logsigmoid(x) = min(x, 0) - log1p(exp(-|x|))
 __global__ void gla_decay_kernel(float* __restrict__ z, const float* __restrict__ bias, long long total, int width, float inv_tau) {
@@ -83,6 +60,8 @@ __global__ void forget_gates_kernel(const float* __restrict__ proj, long long st
     decay[idx] = l + (1.0f - l) * sig;
 }
 
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+
 // ROWS floats from 8- or 16-byte aligned shared memory
 template <int ROWS>
 __device__ __forceinline__ void load_rows(const float* p, float (&v)[ROWS]) {
@@ -98,7 +77,9 @@ __device__ __forceinline__ void load_rows(const float* p, float (&v)[ROWS]) {
     }
 }
 
-template <int ROWS>       // rows of a column one thread holds, side by side: a block's slab has DP = 8 * ROWS rows
+// rows of a column one thread holds, side by side: a block's slab has DP = 8 * ROWS rows.  SILU: q, k and v pass SiLU on
+// their way into shared memory (behind the wait for their loads, not in front of it).
+template <int ROWS, bool SILU>
 __global__ void __launch_bounds__(GLA_THREADS)
 gla_walk_kernel(GlaArgs a) {
     constexpr int DP = 8 * ROWS;
@@ -125,6 +106,7 @@ gla_walk_kernel(GlaArgs a) {
             S[c][i] = (col + c < vdim && row < dim) ? S_base[(long long)(col + c) * dim + row] : 0.0f;
         }
 
+    const float const_decay = a.const_decay != nullptr ? a.const_decay[head] : 1.0f;
     float rq[U], rk[U], ra[U], rv[GLA_V_LOADS];
     auto fetch = [&](int c0) {
         const int n_here = min(GLA_CHUNK, t1 - c0);
@@ -138,15 +120,18 @@ gla_walk_kernel(GlaArgs a) {
                 const float* row = a.qk + (long long)(c0 + tt) * a.qk_stride + (head / a.qk_share) * dim + row0 + d;
                 rq[u] = row[a.q_col];
                 rk[u] = row[a.k_col];
-                ra[u] = a.head_decay != nullptr ? a.head_decay[(long long)(c0 + tt) * a.H + head]
-                                                : a.decay[(long long)(c0 + tt) * a.H * dim + head * dim + row0 + d];
+                ra[u] = a.const_decay != nullptr ? const_decay
+                        : a.head_decay != nullptr ? a.head_decay[(long long)(c0 + tt) * a.H + head]
+                                                  : a.decay[(long long)(c0 + tt) * a.H * dim + head * dim + row0 + d];
             }
         }
 #pragma unroll
         for (int u = 0; u < GLA_V_LOADS; ++u) {
             const int idx = tid + u * GLA_THREADS;
             const int tt = idx / GLA_COLS, cc = idx % GLA_COLS;
-            rv[u] = (tt < n_here && col0 + cc < vdim) ? a.vsrc[(long long)(c0 + tt) * a.v_stride + a.v_col + head * vdim + col0 + cc] : 0.0f;
+            rv[u] = 0.0f;
+            if (tt < n_here && col0 + cc < a.v_cols) rv[u] = a.vsrc[(long long)(c0 + tt) * a.v_stride + a.v_col + head * a.v_cols + col0 + cc];
+            else if (tt < n_here && col0 + cc < vdim) rv[u] = 1.0f;              // a column of ones behind the head's values
             if (a.v_scale != nullptr && tt < n_here) rv[u] *= a.v_scale[(long long)(c0 + tt) * a.H + head];
         }
     };
@@ -157,12 +142,12 @@ gla_walk_kernel(GlaArgs a) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             const int idx = tid + u * GLA_THREADS;
-            qs[idx] = rq[u] * a.q_scale;
-            ks[idx] = rk[u];
+            qs[idx] = (SILU ? silu_f(rq[u]) : rq[u]) * a.q_scale;
+            ks[idx] = SILU ? silu_f(rk[u]) : rk[u];
             as[idx] = ra[u];
         }
 #pragma unroll
-        for (int u = 0; u < GLA_V_LOADS; ++u) vs[tid + u * GLA_THREADS] = rv[u];
+        for (int u = 0; u < GLA_V_LOADS; ++u) vs[tid + u * GLA_THREADS] = SILU ? silu_f(rv[u]) : rv[u];
         __syncthreads();
         if (c0 + GLA_CHUNK < t1) fetch(c0 + GLA_CHUNK);       // in flight while this chunk is walked
         // groups of four tokens (a single token, a decode step, is a group of one)
@@ -268,19 +253,37 @@ __global__ void state_space_finish_kernel(const float* __restrict__ o, int slice
     }
 }
 
-template <int ROWS>
+template <int ROWS, bool SILU>
 static int launch_gla(const GlaArgs& a, dim3 grid, cudaStream_t s) {
     constexpr int DP = 8 * ROWS;
     const size_t smem = (size_t)(3 * GLA_CHUNK * DP + GLA_CHUNK * GLA_COLS) * sizeof(float);
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
-        cudaError_t e = cudaFuncSetAttribute(gla_walk_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gla_walk_kernel<ROWS, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         raised = true;
     }
-    gla_walk_kernel<ROWS><<<grid, GLA_THREADS, smem, s>>>(a);
+    gla_walk_kernel<ROWS, SILU><<<grid, GLA_THREADS, smem, s>>>(a);
     MLC_LAUNCH_CHECK();
     return 0;
+}
+
+int gla_walk(GlaArgs a, int n_seqs, int n_tokens, int rows, bool silu, cudaStream_t s) {
+    if (a.H <= 0 || a.dim <= 0 || a.dim > 256 || a.vdim <= 0 || a.v_cols <= 0 || a.v_cols > a.vdim || n_seqs > 65535 ||
+        a.qk_share < 1 || a.H % a.qk_share)
+        return MLC_ERR_BAD_SIZE;
+    if (silu && (a.v_scale != nullptr || a.v_cols != a.vdim)) return MLC_ERR_UNSUPPORTED;      // SiLU would act on the scaled v
+    if (rows != 2 && rows != 4 && rows != 8 && rows != 16 && rows != 32) return MLC_ERR_BAD_SIZE;
+    a.col_slabs = (a.vdim + GLA_COLS - 1) / GLA_COLS;
+    a.out_slice = (long long)n_tokens * a.H * a.vdim;
+    const dim3 grid(a.H, n_seqs, a.col_slabs * ((a.dim + 8 * rows - 1) / (8 * rows)));
+#define MLC_GLA_ROWS(R) (silu ? launch_gla<R, true>(a, grid, s) : launch_gla<R, false>(a, grid, s))
+    if (rows == 2) return MLC_GLA_ROWS(2);
+    if (rows == 4) return MLC_GLA_ROWS(4);
+    if (rows == 8) return MLC_GLA_ROWS(8);
+    if (rows == 16) return MLC_GLA_ROWS(16);
+    return MLC_GLA_ROWS(32);
+#undef MLC_GLA_ROWS
 }
 
 }  // namespace mlc
@@ -298,23 +301,18 @@ extern "C" int mlc_gla_rows(int n_seqs, int H, int dim, int vdim, int n_sms) {
     return rows;
 }
 
-// The walk alone, over decays that are already made: q and k (H x dim each) in the float32 rows `qk`, v (H x vdim) in the rows
-// `v` (the same matrix or another), decay float32 [n][H*dim].
-static int gla_walk(const float* qk, long long qk_stride, int q_col, int k_col, const float* v, long long v_stride, int v_col,
-                    const float* decay, float q_scale, float* state, long long state_stride, const int* slots,
-                    const int* cu_seqlens, int n_seqs, int n_tokens, int H, int dim, int vdim, int rows, float* out,
-                    cudaStream_t s, int qk_share = 1, const float* head_decay = nullptr, const float* v_scale = nullptr) {
-    if (H <= 0 || dim <= 0 || dim > 256 || vdim <= 0 || n_seqs > 65535 || qk_share < 1 || H % qk_share) return MLC_ERR_BAD_SIZE;
-    if (rows != 2 && rows != 4 && rows != 8 && rows != 16 && rows != 32) return MLC_ERR_BAD_SIZE;
-    const int col_slabs = (vdim + GLA_COLS - 1) / GLA_COLS, row_slabs = (dim + 8 * rows - 1) / (8 * rows);
-    GlaArgs a{qk, qk_stride, v, v_stride, q_col, k_col, v_col, decay, q_scale, state, state_stride,
-              slots, cu_seqlens, out, (long long)n_tokens * H * vdim, H, dim, vdim, col_slabs, qk_share, head_decay, v_scale};
-    const dim3 grid(H, n_seqs, col_slabs * row_slabs);
-    if (rows == 2) return launch_gla<2>(a, grid, s);
-    if (rows == 4) return launch_gla<4>(a, grid, s);
-    if (rows == 8) return launch_gla<8>(a, grid, s);
-    if (rows == 16) return launch_gla<16>(a, grid, s);
-    return launch_gla<32>(a, grid, s);
+// The walk over one decay per token, head and key channel, or over the state-space layer's (one per token and head).
+static int walk_over(const float* qk, long long qk_stride, int q_col, int k_col, const float* v, long long v_stride, int v_col,
+                     const float* decay, float q_scale, float* state, long long state_stride, const int* slots,
+                     const int* cu_seqlens, int n_seqs, int n_tokens, int H, int dim, int vdim, int rows, float* out,
+                     cudaStream_t s, int qk_share = 1, const float* head_decay = nullptr, const float* v_scale = nullptr) {
+    GlaArgs a = {};
+    a.qk = qk; a.qk_stride = qk_stride; a.q_col = q_col; a.k_col = k_col;
+    a.vsrc = v; a.v_stride = v_stride; a.v_col = v_col;
+    a.decay = decay; a.head_decay = head_decay; a.v_scale = v_scale; a.q_scale = q_scale;
+    a.state = state; a.state_stride = state_stride; a.slots = slots; a.cu_seqlens = cu_seqlens; a.out = out;
+    a.H = H; a.dim = dim; a.vdim = a.v_cols = vdim; a.qk_share = qk_share;
+    return gla_walk(a, n_seqs, n_tokens, rows, false, s);
 }
 
 // proj: float32 rows (stride proj_stride) holding q (H x dim) at q_col, k (H x dim) at k_col, v (H x vdim) at v_col.
@@ -332,8 +330,8 @@ extern "C" int mlc_gla(const float* proj, long long proj_stride, int q_col, int 
     const long long total = (long long)n_tokens * H * dim;
     gla_decay_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(z, z_bias, total, H * dim, 1.0f / tau);
     MLC_LAUNCH_CHECK();
-    return gla_walk(proj, proj_stride, q_col, k_col, proj, proj_stride, v_col, z, 1.0f / sqrtf((float)dim), state, state_stride,
-                    slots, cu_seqlens, n_seqs, n_tokens, H, dim, vdim, rows, out, s);
+    return walk_over(proj, proj_stride, q_col, k_col, proj, proj_stride, v_col, z, 1.0f / sqrtf((float)dim), state, state_stride,
+                     slots, cu_seqlens, n_seqs, n_tokens, H, dim, vdim, rows, out, s);
 }
 
 // The forget-gate form: proj float32 rows holding the query logits (H x dim) at q_col, the gate logits (H x dim) at f_col
@@ -351,7 +349,7 @@ extern "C" int mlc_forget_gate_attention(const float* proj, long long proj_strid
     forget_gates_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(proj, proj_stride, q_col, f_col, f_bias, lower, total,
                                                                          width, qk, decay);
     MLC_LAUNCH_CHECK();
-    return gla_walk(qk, 2LL * width, 0, width, proj, proj_stride, v_col, decay, 1.0f, state, state_stride, slots, cu_seqlens,
+    return walk_over(qk, 2LL * width, 0, width, proj, proj_stride, v_col, decay, 1.0f, state, state_stride, slots, cu_seqlens,
                     n_seqs, n_tokens, H, dim, vdim, rows, out, s);
 }
 
@@ -373,7 +371,7 @@ extern "C" int mlc_state_space(const float* proj, long long proj_stride, int z_c
     const long long total = (long long)n_tokens * H;
     state_space_steps_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(proj, proj_stride, dt_col, dt_bias, A_log, total, H, dt, decay);
     MLC_LAUNCH_CHECK();
-    const int rc = gla_walk(xbc, xbc_stride, c_col, b_col, xbc, xbc_stride, 0, nullptr, 1.0f, state, state_stride, slots, cu_seqlens,
+    const int rc = walk_over(xbc, xbc_stride, c_col, b_col, xbc, xbc_stride, 0, nullptr, 1.0f, state, state_stride, slots, cu_seqlens,
                             n_seqs, n_tokens, H, N, vdim, rows, walk, s, H / G, decay, dt);
     if (rc != 0) return rc;
     const int slices = (N + 8 * rows - 1) / (8 * rows);

@@ -261,13 +261,18 @@ moe_route_scored_kernel(const TX* __restrict__ x, const float* __restrict__ w, c
     if (lane < top) weights[(long long)t * top + lane] = mine / (total + 1e-20f) * scale;
 }
 
+// The pairs' experts are `ids` [n][top], or, when `table` [vocab][top] is given, the row of the table that the token's id
+// names: routing by token identity, which needs no scores.  `weights`, if given, receives `weight` for every pair.
+//
 // One block of 32 warps.  Warp w takes the w-th stretch of the pairs.  Shared: cnt[w][e], the pairs of expert e in
 // stretch w, turned into the row at which stretch w's pairs of expert e begin; inside a stretch the pairs of an expert
 // keep their order (lanes that hold the same expert find each other with match.any), so an expert's rows are its pairs in
 // pair order, whatever the number of warps.
 __global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int top, int E, int tile, int max_rows, int* __restrict__ row_of,
+moe_plan_kernel(const int* __restrict__ ids, const int* __restrict__ tokens, const int* __restrict__ table, float weight,
+                float* __restrict__ weights, int n_pairs, int top, int E, int tile, int max_rows, int* __restrict__ row_of,
                 int* __restrict__ src_tok, int* __restrict__ tile_expert) {
+    auto expert_of = [&](int p) { return table != nullptr ? table[(long long)tokens[p / top] * top + p % top] : ids[p]; };
     extern __shared__ int sh[];
     int* cnt = sh;                 // [32][E]
     int* start = sh + 32 * E;      // [E]: first row of the expert's run
@@ -282,8 +287,10 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int top, int E, int ti
     // row_of is -1
     for (int p0 = p_begin; p0 < p_end; p0 += 32) {
         const int p = p0 + lane;
-        const bool have = p < p_end && ids[p] < E;
-        const int e = have ? ids[p] : -1 - lane;                     // lanes without a pair match nobody
+        const int mine = p < p_end ? expert_of(p) : E;
+        const bool have = mine < E;
+        if (p < p_end && weights != nullptr) weights[p] = weight;
+        const int e = have ? mine : -1 - lane;                       // lanes without a pair match nobody
         const unsigned same = __match_any_sync(0xffffffffu, e);
         if (have && (same & ((1u << lane) - 1u)) == 0) cnt[warp * E + e] += __popc(same);      // the first lane of each expert
         __syncwarp();
@@ -307,9 +314,10 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int top, int E, int ti
     __syncthreads();
     for (int p0 = p_begin; p0 < p_end; p0 += 32) {
         const int p = p0 + lane;
-        const bool have = p < p_end && ids[p] < E;
+        const int mine = p < p_end ? expert_of(p) : E;
+        const bool have = mine < E;
         if (p < p_end && !have) row_of[p] = -1;
-        const int e = have ? ids[p] : -1 - lane;
+        const int e = have ? mine : -1 - lane;
         const unsigned same = __match_any_sync(0xffffffffu, e);
         if (have) {
             const int row = cnt[warp * E + e] + __popc(same & ((1u << lane) - 1u));
@@ -533,17 +541,29 @@ extern "C" int mlc_moe_route_scored(const void* x, int x_dtype, const float* w, 
     return 0;
 }
 
-extern "C" int mlc_moe_plan(const int* ids, int n_pairs, int top, int E, int tile, int max_rows, int* row_of, int* src_tok,
-                            int* tile_expert, void* stream) {
+static int launch_plan(const int* ids, const int* tokens, const int* table, float weight, float* weights, int n_pairs, int top,
+                       int E, int tile, int max_rows, int* row_of, int* src_tok, int* tile_expert, void* stream) {
     if (n_pairs <= 0) return 0;
     if (E <= 0 || E > 256 || tile <= 0 || max_rows % tile != 0 || top <= 0) return MLC_ERR_BAD_SIZE;
     // every expert's run, rounded up to whole tiles, must fit
     const long long most = (long long)n_pairs + (long long)(E < n_pairs ? E : n_pairs) * (tile - 1);     // only experts that were chosen have a run
     if ((long long)max_rows < most - most % tile) return MLC_ERR_BAD_SIZE;
-    moe_plan_kernel<<<1, 1024, 33 * E * sizeof(int), (cudaStream_t)stream>>>(ids, n_pairs, top, E, tile, max_rows, row_of,
-                                                                            src_tok, tile_expert);
+    moe_plan_kernel<<<1, 1024, 33 * E * sizeof(int), (cudaStream_t)stream>>>(ids, tokens, table, weight, weights, n_pairs, top, E, tile,
+                                                                            max_rows, row_of, src_tok, tile_expert);
     MLC_LAUNCH_CHECK();
     return 0;
+}
+
+extern "C" int mlc_moe_plan(const int* ids, int n_pairs, int top, int E, int tile, int max_rows, int* row_of, int* src_tok,
+                            int* tile_expert, void* stream) {
+    return launch_plan(ids, nullptr, nullptr, 0.0f, nullptr, n_pairs, top, E, tile, max_rows, row_of, src_tok, tile_expert, stream);
+}
+
+// The plan of experts chosen by token id: tokens int32 [n] name rows of table int32 [vocab][top], whose entries are below E;
+// weights float32 [n][top] receives `weight` for every pair.
+extern "C" int mlc_moe_plan_table(const int* tokens, const int* table, float weight, float* weights, int n, int top, int E, int tile,
+                                  int max_rows, int* row_of, int* src_tok, int* tile_expert, void* stream) {
+    return launch_plan(nullptr, tokens, table, weight, weights, n * top, top, E, tile, max_rows, row_of, src_tok, tile_expert, stream);
 }
 
 extern "C" int mlc_grouped_linear(const void* x, int x_dtype, const int* src_tok, const void* w, int w_dtype,

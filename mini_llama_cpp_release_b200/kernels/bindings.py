@@ -21,6 +21,7 @@ __all__ = [
     "head_project", "gemm_tcgen05_grouped", "GROUPED_TILE",
     "group_norm", "activation", "forget_gate_attention", "moe_route_scored",
     "tanh_norm", "glu", "sigmoid_gate", "state_space",
+    "decay_attention", "matrix_memory", "rms_pair", "embed_rms", "diff_combine", "moe_plan_table",
 ]
 
 
@@ -95,7 +96,7 @@ def core() -> ctypes.CDLL:
             "mlc_add_rmsnorm": [P, P, I, P, F, I, I, P, I, P],
             "mlc_rope_table": [P, I, I, F, P, P],
             "mlc_layernorm": [P, P, I, P, P, P, I, P, P, F, I, I, I, P, I, P],
-            "mlc_qk_norm_rope_cache": [P, LL, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P, P, LL, I, I, I, P, P, P, I, I, F, I, P],
+            "mlc_qk_norm_rope_cache": [P, LL, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P, P, LL, I, I, I, P, P, P, I, I, F, I, I, P],
             "mlc_softcap": [P, LL, F, P],
             "mlc_causal_conv": [P, LL, P, P, P, I, I, I, P, LL, P, P, P, I, I, I, P, LL, P],
             "mlc_gated_delta_rule": [P, LL, I, I, I, P, LL, I, I, P, P, P, P, LL, P, P, I, I, I, I, I, I, I, P, P],
@@ -110,6 +111,12 @@ def core() -> ctypes.CDLL:
             "mlc_attention_simt": [P, P, I, P, P, I, I, I, I, I, I, F, I, I, P, P, P, P, P, LL, I, I, P, I, I, F, P],
             "mlc_moe_route": [P, I, P, P, I, I, I, I, I, P, P, P],
             "mlc_moe_plan": [P, I, I, I, I, I, P, P, P, P],
+            "mlc_moe_plan_table": [P, P, F, P, I, I, I, I, I, P, P, P, P],
+            "mlc_decay_attention": [P, LL, I, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, I, I, P, P, I, P],
+            "mlc_matrix_memory": [P, LL, I, I, I, I, I, I, P, P, F, P, F, P, LL, P, P, I, I, I, I, I, I, I, P, P, P, I, P],
+            "mlc_rms_pair": [P, P, I, P, P, P, I, P, P, F, I, I, P, P, I, P],
+            "mlc_embed_rms": [P, I, P, I, I, F, P, F, P, P],
+            "mlc_diff_combine": [P, I, P, LL, F, F, F, I, I, I, I, P, P],
             "mlc_grouped_linear": [P, I, P, P, I, P, I, I, I, I, P, I, P],
             "mlc_moe_gather": [P, I, P, I, I, P, P, P, I, P],
             "mlc_moe_combine": [P, P, P, P, I, I, I, I, P, P],
@@ -204,6 +211,16 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: floa
     assert ids.dtype == torch.int32 and ids.numel() == n and table.shape[1] == d and out.dtype == torch.float32
     _check(core().mlc_embed(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), n, d, float(scale), out.data_ptr(), _stream()),
            "embedding")
+
+
+def embed_rms(table: torch.Tensor, ids: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] = v / sqrt(mean(v²) + eps) · gain, v = table[ids[t]] · scale, float32."""
+    require_cuda(table, ids, gain, out)
+    n, d = out.shape
+    assert ids.dtype == torch.int32 and ids.numel() == n and table.shape[1] == d and out.dtype == torch.float32
+    assert gain.dtype == torch.float32 and gain.numel() == d
+    _check(core().mlc_embed_rms(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), n, d, float(scale), gain.data_ptr(),
+                                float(eps), out.data_ptr(), _stream()), "embedding and norm")
 
 
 def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
@@ -403,25 +420,66 @@ def layernorm(x: torch.Tensor, y: Optional[torch.Tensor], gain: torch.Tensor, ep
                                 dtype_code(out.dtype) if out is not None else 0, _stream()), "layer norm")
 
 
+def rms_pair(x: torch.Tensor, gain1: torch.Tensor, gain2: Optional[torch.Tensor], eps: float, out1: torch.Tensor,
+             out2: Optional[torch.Tensor], y: Optional[torch.Tensor] = None, expert_rows=None) -> None:
+    """x (float32 [n, d], in place) += y (float32 [n, d] or slices [s, n, d] that are added up) + the weighted sum of each
+    token's `expert_rows` = (rows, row_of, weights), as far as they are given; then out1 = x / rms(x) · gain1 and, with
+    gain2, out2 = x / rms(x) · gain2 (one root mean square, eps inside the root; both outputs of one type)."""
+    require_cuda(x, gain1, gain2, out1, out2, y)
+    n, d = x.shape
+    assert x.dtype == torch.float32 and tuple(out1.shape) == (n, d) and (gain2 is None) == (out2 is None)
+    assert out2 is None or (out2.dtype == out1.dtype and tuple(out2.shape) == (n, d))
+    for g in (gain1, gain2):
+        assert g is None or (g.dtype == torch.float32 and g.numel() == d)
+    rows, row_of, weights, top = _expert_rows(expert_rows, n, d)
+    n_slices = 1
+    if y is not None:
+        assert y.dtype == torch.float32 and tuple(y.shape[-2:]) == (n, d)
+        n_slices = y.shape[0] if y.dim() == 3 else 1
+    _check(core().mlc_rms_pair(x.data_ptr(), _ptr(y), n_slices, _ptr(rows), _ptr(row_of), _ptr(weights), top, gain1.data_ptr(),
+                               _ptr(gain2), float(eps), n, d, out1.data_ptr(), _ptr(out2), dtype_code(out1.dtype), _stream()),
+           "pair of norms")
+
+
+def diff_combine(o: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, lam: float, eps: float, mult: float, heads: int,
+                 vdim: int, out: torch.Tensor) -> None:
+    """o [n, heads * 2 * D]: each head's two outputs (vdim entries, rows of D); u = o1 - lam · o2,
+    out[t, h] = u / sqrt(mean(u²) + eps) · mult · sigmoid(gate[t, gate_col + h]) (gate float32 rows; None: no gate),
+    out [n, heads * vdim] of o's type."""
+    require_cuda(o, out)
+    n = o.shape[0]
+    D = o.shape[1] // (2 * heads)
+    assert o.shape[1] == 2 * heads * D and D >= vdim and tuple(out.shape) == (n, heads * vdim) and out.dtype == o.dtype
+    if gate is not None:
+        _require_rows(gate)
+    _check(core().mlc_diff_combine(o.data_ptr(), dtype_code(o.dtype), _columns(gate, gate_col) if gate is not None else None,
+                                   gate.stride(0) if gate is not None else 0, float(lam), float(eps), float(mult), n, heads, vdim, D,
+                                   out.data_ptr(), _stream()), "difference of two attention maps")
+
+
 def qk_norm_rope_cache(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_gain: Optional[torch.Tensor],
                        k_gain: Optional[torch.Tensor], eps: float, positions: torch.Tensor, tok_seq: torch.Tensor,
                        rope: Optional[torch.Tensor], rot_dims: int, q_heads: int, kv_heads_in_row: int, dim: int, vdim: int,
                        v_scale: float, q_out: torch.Tensor, kv: Optional[KVView], q_bias: Optional[torch.Tensor] = None,
                        k_bias: Optional[torch.Tensor] = None, v_bias: Optional[torch.Tensor] = None, whole_row: bool = False,
-                       interleaved: bool = False, q_temp: Optional[Tuple[float, int]] = None) -> None:
+                       interleaved: bool = False, q_temp: Optional[Tuple[float, int]] = None, maps: int = 1) -> None:
     """Rows of a float32 projection (q heads at column q_col, k heads at k_col, v heads at v_col): per-head RMS norm of q
     and k (gain optional; a negative eps: none), rotation of the first `rot_dims` entries of each head by the table
     `rope` [positions, rot_dims/2, 2], v times `v_scale`; q into q_out [n, q_heads, D], k and v into the cache, whose
     heads have D >= max(dim, vdim) entries (the rest zero).  Biases (float32, as long as their projections) are added as the
     columns are read.  `whole_row`: one statistic over all q heads and one over all k heads, gains as long as the
     projections.  `interleaved`: the rotation pairs entry 2j with 2j + 1 instead of j with j + rot_dims/2.  `q_temp` =
-    (coef, every): the queries of position p are multiplied by 1 + coef · ln(floor((p + 1) / every) + 1)."""
+    (coef, every): the queries of position p are multiplied by 1 + coef · ln(floor((p + 1) / every) + 1).  `maps` > 1: a key
+    head holds that many keys of `dim` entries side by side (D >= maps * dim), each normed and rotated by itself; of the
+    `q_heads` query heads (maps per head, in order) the h-th meets only key h % maps: its entries stand at that key's place
+    in its row of D, zeros elsewhere."""
     coef, every = q_temp if q_temp is not None else (0.0, 0)
     assert every >= 0
     require_cuda(proj, q_gain, k_gain, positions, tok_seq, rope, q_out, q_bias, k_bias, v_bias)
     for g, heads in ((q_gain, q_heads), (k_gain, kv_heads_in_row)):
         assert g is None or not heads or g.numel() == (heads * dim if whole_row else dim)
-    for b, size in ((q_bias, q_heads * dim), (k_bias, kv_heads_in_row * dim), (v_bias, kv_heads_in_row * vdim)):
+    assert maps >= 1 and q_heads % maps == 0 and (maps == 1 or not whole_row)
+    for b, size in ((q_bias, q_heads * dim), (k_bias, kv_heads_in_row * maps * dim), (v_bias, kv_heads_in_row * vdim)):
         assert b is None or not size or (b.dtype == torch.float32 and b.numel() == size)
     n = proj.shape[0]
     assert proj.dtype == torch.float32 and proj.dim() == 2
@@ -439,7 +497,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
                                          rope.shape[0] if rope is not None else 0, rot_dims if rope is not None else 0, n,
                                          q_heads, kv_heads_in_row, dim, vdim, D, float(v_scale), q_out.data_ptr(),
                                          dtype_code(q_out.dtype), *args, _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
-                                         1 if whole_row else 0, 1 if interleaved else 0, float(coef), int(every), _stream()),
+                                         1 if whole_row else 0, 1 if interleaved else 0, float(coef), int(every), int(maps), _stream()),
            "q/k norm, rotation and cache write")
 
 
@@ -622,6 +680,21 @@ def moe_plan(ids: torch.Tensor, n_experts: int, tile: int, row_of: torch.Tensor,
                                src_tok.data_ptr(), tile_expert.data_ptr(), _stream()), "expert plan")
 
 
+def moe_plan_table(tokens: torch.Tensor, table: torch.Tensor, weight: float, weights: torch.Tensor, n_experts: int, tile: int,
+                   row_of: torch.Tensor, src_tok: torch.Tensor, tile_expert: torch.Tensor) -> None:
+    """`moe_plan` for experts chosen by token id: token t's experts are table[tokens[t]] (int32 [vocab, top], entries below
+    `n_experts`); weights float32 [n, top] receives `weight` everywhere."""
+    require_cuda(tokens, table, weights, row_of, src_tok, tile_expert)
+    n, top = row_of.shape
+    assert tokens.dtype == table.dtype == row_of.dtype == src_tok.dtype == tile_expert.dtype == torch.int32
+    assert tokens.numel() == n and table.shape[1] == top and weights.dtype == torch.float32 and weights.shape == row_of.shape
+    rows = src_tok.numel()
+    assert rows % tile == 0 and tile_expert.numel() == rows // tile
+    _check(core().mlc_moe_plan_table(tokens.data_ptr(), table.data_ptr(), float(weight), weights.data_ptr(), n, top, int(n_experts),
+                                     int(tile), rows, row_of.data_ptr(), src_tok.data_ptr(), tile_expert.data_ptr(), _stream()),
+           "expert plan by token id")
+
+
 def grouped_linear(x: torch.Tensor, src_tok: Optional[torch.Tensor], w: torch.Tensor, tile_expert: torch.Tensor, tile: int,
                    out: torch.Tensor) -> None:
     """out[row] = w[expert of the row's tile] · x[src_tok[row]] (x[row] without src_tok), float32 multiply-adds;
@@ -796,6 +869,57 @@ def state_space(proj: torch.Tensor, z_col: int, dt_col: int, xbc: torch.Tensor, 
                                dt.data_ptr(), decay.data_ptr(), state.data_ptr(), state.stride(0), step.slots.data_ptr(),
                                step.cu_seqlens.data_ptr(), step.n_seqs, n, heads, groups, n_state, vdim, rows, walk.data_ptr(),
                                out.data_ptr(), dtype_code(out.dtype), _stream()), "state-space layer")
+    count_launches(2)
+
+
+# ------------------------------------------------------------------ memories that decay per head (csrc/matrix_memory.cu)
+def decay_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_col: int, decay: torch.Tensor, gain: torch.Tensor,
+                    eps: float, out_scale: float, state: torch.Tensor, step, heads: int, dim: int, vdim: int, out: torch.Tensor) -> None:
+    """Linear attention with one constant decay per head over the step's tokens: S <- decay S + silu(k) silu(v)T,
+    o = ST silu(q); then all heads together divided by their root mean square, times `gain`, times sigmoid(gate), times
+    `out_scale`.  q, k (heads x dim), v and the gate (heads x vdim) in the float32 rows `proj`; decay float32 [heads]; gain float32
+    [heads*vdim]; state float32 [slots, heads*vdim*dim]; out [n, heads*vdim] in the engine's type."""
+    require_cuda(decay, gain, out)
+    _require_rows(state)
+    _require_rows(proj)
+    n = proj.shape[0]
+    lib = core()
+    rows = lib.mlc_gla_rows(step.n_seqs, heads, dim, vdim, _sm_count(out.device))
+    slices = (dim + 8 * rows - 1) // (8 * rows)
+    assert decay.dtype == gain.dtype == torch.float32 and decay.numel() == heads and gain.numel() == heads * vdim
+    assert state.shape[1] == heads * vdim * dim and tuple(out.shape) == (n, heads * vdim)
+    walk = torch.empty(slices * n * heads * vdim, dtype=torch.float32, device=out.device)
+    _check(lib.mlc_decay_attention(proj.data_ptr(), proj.stride(0), q_col, k_col, v_col, g_col, decay.data_ptr(), gain.data_ptr(),
+                                   float(eps), float(out_scale), state.data_ptr(), state.stride(0), step.slots.data_ptr(),
+                                   step.cu_seqlens.data_ptr(), step.n_seqs, n, heads, dim, vdim, rows, walk.data_ptr(),
+                                   out.data_ptr(), dtype_code(out.dtype), _stream()), "linear attention with a constant decay")
+    count_launches(1)
+
+
+def matrix_memory(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_col: int, i_col: int, f_col: int, i_bias: torch.Tensor,
+                  f_bias: torch.Tensor, cap: float, gain: torch.Tensor, eps: float, state: torch.Tensor, step, heads: int, dim: int,
+                  vdim: int, out: torch.Tensor) -> None:
+    """The matrix memory with exponential gates over the step's tokens (csrc/matrix_memory.cu): log gates
+    i = cap·tanh((z_i + i_bias)/cap), f = logsigmoid(cap·tanh((z_f + f_bias)/cap)), a running maximum m, o = ST q dim^-1/2
+    over max(|n·q|, exp(-m)) + 1e-6, per-head RMS norm, times `gain`, times sigmoid(gate).  q, k (heads x dim), v and the
+    output gate (heads x vdim), z_i and z_f (heads) in the float32 rows `proj`; state float32
+    [slots, heads*(vdim+1)*dim + heads]; out [n, heads*vdim] in the engine's type."""
+    require_cuda(i_bias, f_bias, gain, out)
+    _require_rows(state)
+    _require_rows(proj)
+    n = proj.shape[0]
+    lib = core()
+    rows = lib.mlc_gla_rows(step.n_seqs, heads, dim, vdim + 1, _sm_count(out.device))
+    slices = (dim + 8 * rows - 1) // (8 * rows)
+    assert all(t.dtype == torch.float32 for t in (i_bias, f_bias, gain)) and i_bias.numel() == f_bias.numel() == heads
+    assert gain.numel() == heads * vdim and tuple(out.shape) == (n, heads * vdim)
+    assert state.shape[1] == heads * (vdim + 1) * dim + heads
+    scratch = torch.empty(3 * n * heads + slices * n * heads * (vdim + 1), dtype=torch.float32, device=out.device)
+    _check(lib.mlc_matrix_memory(proj.data_ptr(), proj.stride(0), q_col, k_col, v_col, g_col, i_col, f_col, i_bias.data_ptr(),
+                                 f_bias.data_ptr(), float(cap), gain.data_ptr(), float(eps), state.data_ptr(), state.stride(0),
+                                 step.slots.data_ptr(), step.cu_seqlens.data_ptr(), step.n_seqs, n, step.max_q_len, heads, dim,
+                                 vdim, rows, scratch.data_ptr(), scratch[3 * n * heads:].data_ptr(), out.data_ptr(),
+                                 dtype_code(out.dtype), _stream()), "matrix memory with exponential gates")
     count_launches(2)
 
 

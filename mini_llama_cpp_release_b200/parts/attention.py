@@ -396,6 +396,112 @@ class SinkAttention(GQAttention):
         return self._out(self.mix(self.in_proj(h, torch.float32), 0, step, memory), residual)
 
 
+@register_part("mixer", "differential_attention")
+class DifferentialAttention(SinkAttention):
+    """Differential attention (Ye et al., "Differential Transformer"): per head two softmax maps over the same values, of which
+    the second is subtracted from the first.
+
+        q = W_q h + b_q  (heads x 2 x dim),  k = W_k h + b_k  (kv_heads x 2 x dim),  v = W_v h + b_v  (kv_heads x vdim)
+        every map of every q and k head rotated by itself;  a_m = softmax(scale · q_m k_mᵀ, masked) v
+        u = a_1 - lambda · a_2,   lambda = exp(lq1 · lk1) - exp(lq2 · lk2) + diff
+        out = W_o [ u / sqrt(mean(u²) + eps) · (1 - diff) · sigmoid(W_g h)_head ]
+
+    In the cache a key head is the row [map 1 | map 2] and a value head is stored once; a query of map m is a row of the same
+    length with zeros at the other map's place, so its score against the row is the score of its own map.  The attention
+    kernels, which know nothing of this, see 2 · heads query heads on kv_heads key/value heads of
+    D = ceil16(max(2 · dim, vdim)) entries: a step reads every cached key and value once for both maps.
+
+    Options as in `SinkAttention`: `window` and `keep_first`, `bias`, `own_kv`, `keep_all_keys`.  `head_gate`: the sigmoid
+    gate per head (tensor `g`, in the input product).  `names`: the tensors' names below the part's prefix, by role (q, k, v,
+    o, g, lq1, lk1, lq2, lk2; a bias is its matrix's name with `.b`)."""
+    graph_safe = True
+
+    NAMES = dict(q="q", k="k", v="v", o="o", g="g", lq1="lq1", lk1="lk1", lq2="lq2", lk2="lk2")
+    MAPS = 2
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float,
+                 norm_eps: float, diff: float, position: PartSpec, window: Optional[int] = None, keep_first: int = 0, bias: bool = True,
+                 head_gate: bool = True, own_kv: bool = True, keep_all_keys: bool = False, names: Optional[dict] = None):
+        Part.__init__(self, name, hidden_size=hidden_size, num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim,
+                      v_head_dim=v_head_dim, scale=scale, norm_eps=norm_eps, diff=diff, window=window, keep_first=keep_first,
+                      bias=bias, head_gate=head_gate, own_kv=own_kv, keep_all_keys=keep_all_keys)
+        if num_heads % num_kv_heads:
+            raise ValueError(f"attention: {num_heads} query heads are not a multiple of {num_kv_heads} kv heads")
+        self.hidden, self.heads, self.KV = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.H = self.MAPS * self.heads                               # query heads as the attention kernels see them
+        self.dim, self.vdim = int(head_dim), int(v_head_dim)
+        self.hd = (max(self.MAPS * self.dim, self.vdim) + 15) // 16 * 16
+        if self.hd > 512:
+            raise ValueError(f"differential attention: 2 · dim and vdim up to 512 are supported, got dim {head_dim} and vdim {v_head_dim}")
+        if not scale > 0:
+            raise ValueError(f"attention: the score's scale must be positive, got {scale}")
+        self.scale, self.eps, self.diff = float(scale), float(norm_eps), float(diff)
+        self.window = int(window) if window else None
+        self.keep_first = max(0, int(keep_first)) if self.window else 0
+        self.has_bias, self.head_gate, self.own_kv = bool(bias), bool(head_gate), bool(own_kv)
+        self.keep_all_keys = bool(keep_all_keys)
+        self.softcap = self.chunk = self.sinks = None
+        self.t = {role: name + n for role, n in {**self.NAMES, **(names or {})}.items()}
+        self.position = build_part(position, name)
+        self.interleaved = bool(getattr(self.position, "interleaved", False))
+
+    def tensors(self):
+        t, nq, nk = self.t, self.H * self.dim, self.KV * self.MAPS * self.dim
+        specs = [TensorSpec(t["q"], (nq, self.hidden)), TensorSpec(t["o"], (self.hidden, self.heads * self.vdim))]
+        if self.own_kv:
+            specs += [TensorSpec(t["k"], (nk, self.hidden)), TensorSpec(t["v"], (self.KV * self.vdim, self.hidden))]
+        if self.has_bias:
+            specs.append(TensorSpec(t["q"] + ".b", (nq,), role="bias"))
+            if self.own_kv:
+                specs += [TensorSpec(t["k"] + ".b", (nk,), role="bias"), TensorSpec(t["v"] + ".b", (self.KV * self.vdim,), role="bias")]
+        specs += [TensorSpec(t[r], (self.dim,), role="bias") for r in ("lq1", "lk1", "lq2", "lk2")]
+        if self.head_gate:
+            specs.append(TensorSpec(t["g"], (self.heads, self.hidden)))
+        return specs
+
+    def bind(self, get, runtime):
+        Part.bind(self, get, runtime)
+        t = self.t
+        f32 = lambda name: get(name).to(torch.float32).contiguous()
+        # columns of the input product: q | k | v | g (without the parts the mixer does not have)
+        self._in = [get(t["q"])] + ([get(t["k"]), get(t["v"])] if self.own_kv else []) + ([get(t["g"])] if self.head_gate else [])
+        self.in_proj: Optional[Linear] = None
+        self.q_bias = f32(t["q"] + ".b") if self.has_bias else None
+        self.k_bias = f32(t["k"] + ".b") if self.has_bias and self.own_kv else None
+        self.v_bias = f32(t["v"] + ".b") if self.has_bias and self.own_kv else None
+        dot = lambda a, b: float((get(t[a]).double() * get(t[b]).double()).sum().item())           # read once, at load
+        self.lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.diff
+        self.o = Linear(get(t["o"]), runtime)
+        # rows of more than 256 entries run on the float32-arithmetic kernel in both engine types
+        self.use_tensor_cores = runtime.dtype == torch.bfloat16 and self.hd <= 256
+        if self.use_tensor_cores:
+            kernels.attention_library(self.hd)
+
+    def mix(self, proj: torch.Tensor, col: int, step, memory: MixerMemory) -> torch.Tensor:
+        """Attention from the float32 projection rows `proj`, whose columns from `col` on are [q | k | v | g]; returns the
+        heads' outputs [n, heads·vdim] in the engine's type, the input of `self.o`."""
+        rt = self.runtime
+        n = proj.shape[0]
+        if memory.writes_cache != self.own_kv:
+            raise ValueError("attention: a mixer without keys and values of its own reads another run's cache entry, and only "
+                             "such a mixer does")
+        table = self.position.table_for(step.max_kv_len) if hasattr(self.position, "table_for") else None
+        rot = getattr(self.position, "dims", 0) if table is not None else 0
+        q = rt.empty(n, self.H * self.hd)
+        k_col = col + self.H * self.dim
+        v_col = k_col + self.KV * self.MAPS * self.dim
+        g_col = v_col + self.KV * self.vdim if self.own_kv else k_col
+        kernels.qk_norm_rope_cache(proj, col, k_col, v_col, None, None, -1.0, step.positions, step.tok_seq, table, rot, self.H,
+                                   self.KV if self.own_kv else 0, self.dim, self.vdim, 1.0, q, memory.kv if self.own_kv else None,
+                                   q_bias=self.q_bias, k_bias=self.k_bias, v_bias=self.v_bias, interleaved=self.interleaved,
+                                   maps=self.MAPS)
+        o = rt.empty(n, self.H * self.hd)
+        self.attend(q, o, step, memory.kv)
+        act = rt.empty(n, self.heads * self.vdim)
+        kernels.diff_combine(o, proj if self.head_gate else None, g_col, self.lam, self.eps, 1.0 - self.diff, self.heads, self.vdim, act)
+        return act
+
+
 @register_part("mixer", "latent_attention")
 class LatentAttention(GQAttention):
     """Attention whose keys and values are expansions of a low-rank latent (the "multi-head latent attention" of

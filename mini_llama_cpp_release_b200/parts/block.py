@@ -298,6 +298,59 @@ class ParallelBlock(Part):
         return x, None
 
 
+@register_part("block", "parallel_prenorm")
+class ParallelPreNormBlock(Part):
+    """Two norms of the same stream, two branches, one sum: x <- x + (mixer(N1(x)) + feed_forward(N2(x))).  The feed-forward
+    (with its norm) may be absent.
+
+    Both norms are RMS norms of one size and eps (`forward_pair`): one kernel adds what the block before left, forms the root
+    mean square once and writes both branches' inputs.  The branches then add into the stream in their output products'
+    epilogues where they can (`accumulates`), the shared expert of a mixture too; the rows of a mixture's chosen experts are
+    left in the step's `handover` (`DeferredBranch`) for the next block's norm kernel."""
+    graph_safe = True
+    takes_deferred_update = True
+
+    def __init__(self, name: str, mixer: PartSpec, mixer_norm: PartSpec, feed_forward: Optional[PartSpec] = None,
+                 feed_forward_norm: Optional[PartSpec] = None, names: Optional[dict] = None):
+        super().__init__(name)
+        names = names or {}
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("parallel_prenorm block: a feed-forward and its norm come together or not at all")
+        self.mixer_norm = build_part(mixer_norm, name + names.get("mixer_norm", "mixer_norm."))
+        self.mixer = build_part(mixer, name + names.get("mixer", "mixer."))
+        self.feed_forward_norm = (build_part(feed_forward_norm, name + names.get("feed_forward_norm", "feed_forward_norm."))
+                                  if feed_forward_norm else None)
+        self.feed_forward = build_part(feed_forward, name + names.get("feed_forward", "feed_forward.")) if feed_forward else None
+        a, b = self.mixer_norm, self.feed_forward_norm
+        if not hasattr(a, "forward_pair") or (b is not None and (type(a) is not type(b) or a.size != b.size or a.eps != b.eps)):
+            raise ValueError("parallel_prenorm block: its two norms must offer `forward_pair` and have one size and eps")
+
+    def children(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None)
+
+    def forward(self, x: torch.Tensor, pending: Optional[torch.Tensor], step, memory: MixerMemory
+                ) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+        mixer, ff = self.mixer, self.feed_forward
+        left, rows = step.handover.pop(DEFERRED, None), None
+        if left is not None and left.x is x and left.norm is None:
+            rows = left.expert_rows
+        elif left is not None:
+            left.finish()
+        h1, h2 = self.mixer_norm.forward_pair(x, self.feed_forward_norm, pending, rows)
+        y = mixer.forward(h1, step, memory, residual=x) if getattr(mixer, "accumulates", False) else mixer.forward(h1, step, memory)
+        if ff is None:
+            return x, y
+        if hasattr(ff, "forward_shared") and not getattr(ff, "identity", 0) and not getattr(ff, "sum_is_plain", False):
+            s = ff.forward_shared(h2, step, residual=x)
+            step.handover[DEFERRED] = DeferredBranch(x, expert_rows=ff.forward(h2, step, deferred=True))
+        else:
+            s = ff.forward(h2, step, residual=x) if getattr(ff, "accumulates", False) else ff.forward(h2, step)
+        if y is not None and s is not None:
+            kernels.scaled_add(x, y, None, s, None)
+            return x, None
+        return x, y if y is not None else s
+
+
 @register_part("block", "stream_mix")
 class StreamMix(Part):
     """Not a layer but a step between layers: x <- W [x ; e], with e the embedding's output of the step's tokens and W

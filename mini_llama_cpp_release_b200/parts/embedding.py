@@ -8,20 +8,28 @@ from typing import Optional
 import torch
 
 from .. import kernels
-from ..config.registry import register_part
+from ..config.registry import build_part, register_part
+from ..config.specs import PartSpec
 from .base import Part, TensorSpec
 from .linear import Linear
+from .norm import RMSNorm
 
 
 @register_part("embedding", "token_embedding")
 class TokenEmbedding(Part):
     graph_safe = True
 
-    def __init__(self, name: str, vocab_size: int, hidden_size: int, tensor: str = "weight", scale: float = 1.0):
-        """`tensor`: the table's name below the part's prefix.  `scale` multiplies every row as it is read (float32)."""
+    def __init__(self, name: str, vocab_size: int, hidden_size: int, tensor: str = "weight", scale: float = 1.0,
+                 norm: Optional[PartSpec] = None):
+        """`tensor`: the table's name below the part's prefix.  `scale` multiplies every row as it is read (float32).  `norm`: a
+        norm of the embedded rows, whose output is the stream's first value (an RMS norm is part of the gather's kernel)."""
         super().__init__(name, vocab_size=vocab_size, hidden_size=hidden_size, tensor=tensor, scale=scale)
         self.vocab, self.hidden, self.scale = int(vocab_size), int(hidden_size), float(scale)
         self.tensor = self.name + tensor
+        self.norm = build_part(norm, name) if norm is not None else None
+
+    def children(self):
+        return (self.norm,) if self.norm is not None else ()
 
     def tensors(self):
         return [TensorSpec(self.tensor, (self.vocab, self.hidden), role="table")]
@@ -35,8 +43,11 @@ class TokenEmbedding(Part):
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         x = self.runtime.empty(token_ids.numel(), self.hidden, dtype=torch.float32)
+        if isinstance(self.norm, RMSNorm):
+            kernels.embed_rms(self.table, token_ids, self.norm.gain, self.norm.eps, x, self.scale)
+            return x
         kernels.embed(self.table, token_ids, x, self.scale)
-        return x
+        return x if self.norm is None else self.norm.forward(x, out_dtype=torch.float32)
 
 
 @register_part("head", "linear_head")

@@ -9,7 +9,8 @@ from typing import Optional
 import torch
 
 from .. import kernels
-from ..config.registry import register_part
+from ..config.registry import build_part, register_part
+from ..config.specs import PartSpec
 from .base import Part, TensorSpec
 from .linear import Linear
 
@@ -92,6 +93,11 @@ class MixtureOfExperts(Part):
     `weight_scale`.  `identity`: that many further router outputs, behind the experts', belong to identity
     experts, which have no tensors and return their input; they take part in scores, groups and choice like the others.
     `routing="sigmoid"`: s = sigmoid(z); chosen are the `top` largest; the weights are the chosen scores as they are.
+    `routing="table"`: there is no router; a stored table (tensor `table`, integers [vocab, top]) gives every token id its
+    experts, each of weight 1/top.  The plan's kernel reads the table itself.
+
+    `shared`: one more feed-forward that every token passes and whose output is added (a part of its own).  Its output is
+    not part of the rows that a deferring caller adds up: see `forward_shared`.
 
     `weight_on="input"`: a chosen expert's weight multiplies its input, not its output: the output is the plain sum of
     expert(w · h) over the chosen (for experts that are not linear in their input this is another function).
@@ -108,26 +114,31 @@ class MixtureOfExperts(Part):
     graph_safe = True
 
     NAMES = dict(router="router", router_bias="router.b", correction="correction", expert="e{e}.", gate="gate", up="up",
-                 down="down")
+                 down="down", table="table", shared="shared.")
     TILE = 64                        # rows per block of the grouped product; an expert's run is padded to it
 
     def __init__(self, name: str, hidden_size: int, intermediate_size: int, num_experts: int, top: int,
                  router_bias: bool = True, names: Optional[dict] = None, gated: bool = True, activation: str = "silu",
                  routing: str = "top_logits", correction: bool = False, group_count: int = 1, group_keep: int = 1,
                  identity: int = 0, weight_scale: float = 1.0, weight_on: str = "output", limit: Optional[float] = None,
-                 act_alpha: float = 1.0, score: str = "softmax", group_score: str = "max"):
+                 act_alpha: float = 1.0, score: str = "softmax", group_score: str = "max", vocab_size: int = 0,
+                 shared: Optional[PartSpec] = None):
         super().__init__(name, hidden_size=hidden_size, intermediate_size=intermediate_size, num_experts=num_experts, top=top,
                          router_bias=router_bias, gated=gated, activation=activation, routing=routing, correction=correction,
                          group_count=group_count, group_keep=group_keep, identity=identity, weight_scale=weight_scale,
-                         weight_on=weight_on, limit=limit, act_alpha=act_alpha, score=score, group_score=group_score)
+                         weight_on=weight_on, limit=limit, act_alpha=act_alpha, score=score, group_score=group_score,
+                         vocab_size=vocab_size)
         self.hidden, self.inter, self.E, self.top = int(hidden_size), int(intermediate_size), int(num_experts), int(top)
         self.identity = int(identity)
         self.outputs = self.E + self.identity                     # what the router puts out
         if self.E < 1 or self.identity < 0 or not 1 <= self.top <= self.outputs or self.top > 32 or self.outputs > 256:
             raise ValueError(f"mixture of experts: top {top} of {num_experts} experts (+ {identity} identity experts) is not "
                              f"supported (top <= 32, router outputs <= 256)")
-        if routing not in ("top_logits", "scores", "sigmoid"):
-            raise ValueError(f"mixture of experts: routing must be \"top_logits\", \"scores\" or \"sigmoid\", got {routing!r}")
+        if routing not in ("top_logits", "scores", "sigmoid", "table"):
+            raise ValueError(f"mixture of experts: routing must be \"top_logits\", \"scores\", \"sigmoid\" or \"table\", got {routing!r}")
+        self.vocab = int(vocab_size)
+        if routing == "table" and self.vocab < 1:
+            raise ValueError("mixture of experts: routing by a table needs the vocabulary's size")
         if gated and activation not in ("silu", "clamped"):
             raise ValueError(f"mixture of experts: activation {activation!r} is not supported by gated experts")
         if not gated and activation not in kernels.bindings.ACTIVATIONS:
@@ -158,12 +169,19 @@ class MixtureOfExperts(Part):
             if self.group_keep * (self.outputs // self.group_count) < self.top:
                 raise ValueError(f"mixture of experts: {group_keep} groups of {self.outputs // self.group_count} hold fewer than top = {top} experts")
         self.t = {**self.NAMES, **(names or {})}
+        self.shared = build_part(shared, name + self.t["shared"]) if shared is not None else None
+
+    def children(self):
+        return (self.shared,) if self.shared is not None else ()
 
     def _expert(self, e: int, role: str) -> str:
         return self.name + self.t["expert"].format(e=e) + self.t[role]
 
     def tensors(self):
-        specs = [TensorSpec(self.name + self.t["router"], (self.outputs, self.hidden))]
+        if self.routing == "table":
+            specs = [TensorSpec(self.name + self.t["table"], (self.vocab, self.top), role="int_table", init="distinct_rows", below=self.E)]
+        else:
+            specs = [TensorSpec(self.name + self.t["router"], (self.outputs, self.hidden))]
         if self.has_bias:
             specs.append(TensorSpec(self.name + self.t["router_bias"], (self.E,), role="bias"))
         if self.has_correction:
@@ -177,7 +195,14 @@ class MixtureOfExperts(Part):
 
     def bind(self, get, runtime):
         super().bind(get, runtime)
-        self.router = get(self.name + self.t["router"]).to(torch.float32).contiguous()        # the router is float32 in both modes
+        self.router = self.table = None
+        if self.routing == "table":
+            self.table = get(self.name + self.t["table"]).to(torch.int32).contiguous()
+            lo, hi = int(self.table.min()), int(self.table.max())                                # read once, at load
+            if lo < 0 or hi >= self.E:
+                raise ValueError(f"mixture of experts: {self.name + self.t['table']} names experts {lo}..{hi}, but there are {self.E}")
+        else:
+            self.router = get(self.name + self.t["router"]).to(torch.float32).contiguous()    # the router is float32 in both modes
         self.router_bias = get(self.name + self.t["router_bias"]).to(torch.float32).contiguous() if self.has_bias else None
         self.correction = get(self.name + self.t["correction"]).to(torch.float32).contiguous() if self.has_correction else None
         # [E, 2*inter, hidden]: an expert's gate rows, then its up rows (ungated: [E, inter, hidden]); [E, hidden, inter]
@@ -203,11 +228,12 @@ class MixtureOfExperts(Part):
     def weight_bytes(self) -> int:
         """Bytes a step of many tokens reads; a step of few tokens reads `top` experts per token at most."""
         return (self.gate_up.numel() * self.gate_up.element_size() + self.down.numel() * self.down.element_size()
-                + self.router.numel() * 4)
+                + (self.router.numel() * 4 if self.router is not None else 0)
+                + (self.shared.weight_bytes() if self.shared is not None else 0))
 
     def flops_per_token(self) -> float:
         """Multiply-adds x 2 a token costs: the router and `top` experts."""
-        return 2.0 * (self.outputs * self.hidden + self.top * (3 if self.gated else 2) * self.inter * self.hidden)
+        return 2.0 * ((self.outputs * self.hidden if self.router is not None else 0) + self.top * (3 if self.gated else 2) * self.inter * self.hidden)
 
     def route(self, h: torch.Tensor):
         """(ids int32 [n, top], weights float32 [n, top]); an id of `num_experts` or more names an identity expert."""
@@ -224,7 +250,18 @@ class MixtureOfExperts(Part):
                               weighting="sigmoid" if self.routing == "sigmoid" else "softmax")
         return ids, weights
 
-    defers_sum = True         # forward(..., deferred=True) may leave the weighted sum of a token's rows to the caller
+    @property
+    def defers_sum(self) -> bool:
+        """forward(..., deferred=True) may leave the weighted sum of a token's rows to the caller.  With a shared expert only
+        a caller that asks for its output itself (`forward_shared`) may defer."""
+        return self.shared is None
+
+    def forward_shared(self, h: torch.Tensor, step=None, residual: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+        """The shared expert's output, float32 [n, hidden] or slices of it; None if there is none, or if it was added into
+        `residual`."""
+        if self.shared is None:
+            return None
+        return self.shared.forward(h, step, residual=residual)
 
     @property
     def sum_is_plain(self) -> bool:
@@ -238,13 +275,17 @@ class MixtureOfExperts(Part):
         negative row_of stands for the token's own input h (an identity expert)."""
         rt = self.runtime
         n = h.shape[0]
-        ids, weights = self.route(h)
+        by_table = self.routing == "table"
+        ids, weights = (None, rt.empty(n, self.top, dtype=torch.float32)) if by_table else self.route(h)
         tile = kernels.GROUPED_TILE if self.fused else self.TILE
         rows = kernels.moe_plan_rows(n * self.top, self.E, tile)
         row_of = rt.empty(n, self.top, dtype=torch.int32)
         src_tok = rt.empty(rows, dtype=torch.int32)
         tile_expert = rt.empty(rows // tile, dtype=torch.int32)
-        kernels.moe_plan(ids, self.E, tile, row_of, src_tok, tile_expert)
+        if by_table:
+            kernels.moe_plan_table(step.tokens, self.table, 1.0 / self.top, weights, self.E, tile, row_of, src_tok, tile_expert)
+        else:
+            kernels.moe_plan(ids, self.E, tile, row_of, src_tok, tile_expert)
         y = rt.empty(rows, self.hidden, dtype=torch.float32)
         act = rt.empty(rows, self.inter)
         on_input = (weights, row_of) if self.weight_on_input else (None, None)
@@ -276,4 +317,5 @@ class MixtureOfExperts(Part):
             return y, row_of, weights
         out = rt.empty(n, self.hidden, dtype=torch.float32)
         kernels.moe_combine(y, row_of, None if self.weight_on_input else weights, out, ident=h if self.identity else None)
-        return out
+        s = self.forward_shared(h, step)
+        return out if s is None else out.add_(s.sum(dim=0) if s.dim() == 3 else s)

@@ -20,10 +20,12 @@ from .base import Part, TensorSpec
 class RMSNorm(Part):
     graph_safe = True
 
-    def __init__(self, name: str, size: int, eps: float, tensor: str = "weight", offset: float = 0.0):
+    def __init__(self, name: str, size: int, eps: float, tensor: str = "weight", offset: float = 0.0, scale: float = 1.0):
         """`tensor`: the gain's name below the part's prefix.  `offset` is added to the stored values: a gain that is
-        stored around zero and applied as 1 + w has offset 1."""
-        super().__init__(name, size=size, eps=eps, tensor=tensor, offset=offset)
+        stored around zero and applied as 1 + w has offset 1.  `scale` multiplies the gain (a factor on what a linear part
+        without a bias makes of the norm's output)."""
+        super().__init__(name, size=size, eps=eps, tensor=tensor, offset=offset, scale=scale)
+        self.scale = float(scale)
         self.size = int(size)
         self.eps = float(eps)
         self.offset = float(offset)
@@ -34,7 +36,7 @@ class RMSNorm(Part):
 
     def bind(self, get, runtime):
         super().bind(get, runtime)
-        self.gain = (get(self.tensor).to(torch.float32) + self.offset).contiguous()
+        self.gain = ((get(self.tensor).to(torch.float32) + self.offset) * self.scale).contiguous()
 
     def weight_bytes(self) -> int:
         return self.gain.numel() * 4
@@ -45,6 +47,14 @@ class RMSNorm(Part):
         out = self.runtime.empty(*x.shape, dtype=out_dtype or self.runtime.dtype)
         kernels.add_rmsnorm(x, delta, self.gain, self.eps, out)
         return out
+
+    def forward_pair(self, x: torch.Tensor, other: Optional["RMSNorm"], delta: Optional[torch.Tensor] = None, expert_rows=None):
+        """This norm and another of the same size and eps on the same x, which takes `delta` and the weighted sum of
+        `expert_rows` first (see `kernels.rms_pair`); returns both outputs in the engine's type (None for no other)."""
+        out1 = self.runtime.empty(*x.shape)
+        out2 = self.runtime.empty(*x.shape) if other is not None else None
+        kernels.rms_pair(x, self.gain, other.gain if other is not None else None, self.eps, out1, out2, y=delta, expert_rows=expert_rows)
+        return out1, out2
 
 
 @register_part("norm", "layernorm")

@@ -25,6 +25,14 @@ def _f32(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float32).contiguous()
 
 
+def project_out(o: Linear, act: torch.Tensor, residual: Optional[torch.Tensor]):
+    """The output product: added into the stream `residual` if that is given and the product can (returns None)."""
+    if residual is not None and act.dtype == torch.bfloat16 and o.can_add_into_stream(act.shape[0]):
+        o.add_into(act, residual)
+        return None
+    return o(act, torch.float32, partial_ok=True)
+
+
 @register_part("mixer", "gated_delta")
 class GatedDeltaMixer(Part):
     """The gated delta rule (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule").
@@ -272,6 +280,168 @@ class ForgetGateAttention(Part):
         return self.o(self.mix(self.in_proj(h, torch.float32), 0, step, memory), torch.float32, partial_ok=True)
 
 
+@register_part("mixer", "decay_attention")
+class DecayAttention(Part):
+    """Linear attention with one constant decay per head ("Lightning Attention"; Qin et al., "Lightning Attention-2: A Free Lunch
+    for Handling Unlimited Sequence Lengths in Large Language Models").
+
+        q = silu(W_q h), k = silu(W_k h)  (heads x dim);   v = silu(W_v h)  (heads x vdim)
+        S_t = decay_head · S_{t-1} + k_t v_tᵀ;   o_t = S_tᵀ q_t                          (no further scale)
+        out = W_o ( o / rms(o) · w_norm · sigmoid(W_g h) )      (one root mean square over all heads together)
+
+    State per sequence: S for every head, float32, zero at the start.  The walk over tokens is the one of
+    `GatedLinearAttention`.  `out_scale` multiplies the output product's input in float32.  Offers `in_weights()`,
+    `in_width()`, `mix()` and `o`.  `names`: the tensors' names below the part's prefix, by role."""
+    graph_safe = True
+
+    NAMES = dict(q="q", k="k", v="v", g="g", o="o", norm="norm")
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay, norm_eps: float,
+                 out_scale: float = 1.0, names: Optional[dict] = None):
+        super().__init__(name, hidden_size=hidden_size, num_heads=num_heads, head_dim=head_dim, v_head_dim=v_head_dim,
+                         decay=tuple(decay), norm_eps=norm_eps, out_scale=out_scale)
+        self.hidden, self.H, self.dim, self.vdim = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        self.decay_values = [float(d) for d in decay]
+        if len(self.decay_values) != self.H:
+            raise ValueError(f"linear attention: {num_heads} heads need as many decays, got {len(self.decay_values)}")
+        if not 1 <= self.dim <= 256:
+            raise ValueError(f"linear attention: key sizes up to 256 are supported, got {head_dim}")
+        self.n_qk, self.n_v = self.H * self.dim, self.H * self.vdim
+        if self.n_v > 16384:
+            raise ValueError(f"linear attention: up to 16384 value channels are supported, got {self.n_v}")
+        self.eps, self.out_scale = float(norm_eps), float(out_scale)
+        self.t = {role: name + n for role, n in {**self.NAMES, **(names or {})}.items()}
+
+    def tensors(self):
+        t, hid = self.t, self.hidden
+        return [TensorSpec(t["q"], (self.n_qk, hid)), TensorSpec(t["k"], (self.n_qk, hid)), TensorSpec(t["v"], (self.n_v, hid)),
+                TensorSpec(t["g"], (self.n_v, hid)), TensorSpec(t["o"], (hid, self.n_v)),
+                TensorSpec(t["norm"], (self.n_v,), role="gain", init="one_plus_normal")]
+
+    def cache_need(self):
+        return None
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.H * self.vdim * self.dim,), torch.float32)
+
+    def bind(self, get, runtime):
+        super().bind(get, runtime)
+        t = self.t
+        self._in = [get(t[r]) for r in ("q", "k", "v", "g")]     # columns of the input product: q | k | v | g
+        self.in_proj: Optional[Linear] = None
+        self.gain = _f32(get(t["norm"]))
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.gain.device)
+        self.o = Linear(get(t["o"]), runtime)
+
+    def in_weights(self):
+        return list(self._in)
+
+    def in_width(self) -> int:
+        return 2 * self.n_qk + 2 * self.n_v
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in self._in) + self.o.nbytes()
+
+    def mix(self, proj: torch.Tensor, col: int, step, memory: MixerMemory) -> torch.Tensor:
+        """From the float32 projection rows `proj`, whose columns from `col` on are [q | k | v | g]: the normed, gated heads
+        [n, heads·vdim] in the engine's type, the input of `self.o`."""
+        act = self.runtime.empty(proj.shape[0], self.n_v)
+        k_col = col + self.n_qk
+        v_col = k_col + self.n_qk
+        kernels.decay_attention(proj, col, k_col, v_col, v_col + self.n_v, self.decay, self.gain, self.eps, self.out_scale,
+                                memory.state, step, self.H, self.dim, self.vdim, act)
+        return act
+
+    accumulates = True        # forward(..., residual=x) may add the branch into the float32 stream and return None
+
+    def forward(self, h: torch.Tensor, step, memory: MixerMemory, residual: Optional[torch.Tensor] = None):
+        if self.in_proj is None:
+            self.in_proj = fused_rows(self._in, self.runtime)
+        return project_out(self.o, self.mix(self.in_proj(h, torch.float32), 0, step, memory), residual)
+
+
+@register_part("mixer", "matrix_memory")
+class MatrixMemory(Part):
+    """The matrix memory of xLSTM (mLSTM; Beck et al., "xLSTM: Extended Long Short-Term Memory"): an exponential input gate and a
+    sigmoid forget gate per head, both soft-capped, stabilised by a running maximum.
+
+        q = W_q h · dim^-1/2,  k = W_k h  (heads x dim);   v = W_v h  (heads x vdim)
+        i = c · tanh((W_i h + b_i) / c),   f = logsigmoid(c · tanh((W_f h + b_f) / c))            (one per head; c = gate_cap)
+        m_t = max(f + m_{t-1}, i)                                                              (m_0 = 0)
+        S_t = exp(f + m_{t-1} - m_t) S_{t-1} + exp(i - m_t) k vᵀ;   n_t the same with k alone
+        o = S_tᵀ q / (max(|n_t · q|, exp(-m_t)) + 1e-6)
+        out = W_o ( o / rms(o) · w_norm · sigmoid(W_g h) )               (rms over vdim per head, w_norm as long as all heads)
+
+    State per sequence: S and, as one more column of it, n for every head, then every head's m; float32, zero at the start.
+    Gates, m, the recurrence and the norm are float32 in both engine modes.  The walk over tokens is the one of
+    `GatedLinearAttention` with one decay per token and head.  `names`: the tensors' names below the part's prefix, by role."""
+    graph_safe = True
+
+    NAMES = dict(q="q", k="k", v="v", g="g", o="o", norm="norm", i="i", i_bias="i.b", f="f", f_bias="f.b")
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, gate_cap: float, norm_eps: float,
+                 names: Optional[dict] = None):
+        super().__init__(name, hidden_size=hidden_size, num_heads=num_heads, head_dim=head_dim, v_head_dim=v_head_dim,
+                         gate_cap=gate_cap, norm_eps=norm_eps)
+        if not 1 <= head_dim <= 256 or not 1 <= v_head_dim <= 1024:
+            raise ValueError(f"matrix memory: key sizes up to 256 and value sizes up to 1024 are supported, got {head_dim} and {v_head_dim}")
+        if not gate_cap > 0:
+            raise ValueError(f"matrix memory: the gates' cap must be positive, got {gate_cap}")
+        self.hidden, self.H, self.dim, self.vdim = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        self.cap, self.eps = float(gate_cap), float(norm_eps)
+        self.t = {role: name + n for role, n in {**self.NAMES, **(names or {})}.items()}
+        self.n_qk, self.n_v = self.H * self.dim, self.H * self.vdim
+
+    def tensors(self):
+        t, hid = self.t, self.hidden
+        return [TensorSpec(t["q"], (self.n_qk, hid)), TensorSpec(t["k"], (self.n_qk, hid)), TensorSpec(t["v"], (self.n_v, hid)),
+                TensorSpec(t["g"], (self.n_v, hid)), TensorSpec(t["i"], (self.H, hid)), TensorSpec(t["i_bias"], (self.H,), role="bias"),
+                TensorSpec(t["f"], (self.H, hid)), TensorSpec(t["f_bias"], (self.H,), role="bias"),
+                TensorSpec(t["o"], (hid, self.n_v)), TensorSpec(t["norm"], (self.n_v,), role="gain", init="one_plus_normal")]
+
+    def cache_need(self):
+        return None
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((self.H * (self.vdim + 1) * self.dim + self.H,), torch.float32)
+
+    def bind(self, get, runtime):
+        super().bind(get, runtime)
+        t = self.t
+        self._in = [get(t[r]) for r in ("q", "k", "v", "g", "i", "f")]      # columns of the input product, in this order
+        self.in_proj: Optional[Linear] = None
+        self.i_bias, self.f_bias, self.gain = (_f32(get(t[r])) for r in ("i_bias", "f_bias", "norm"))
+        self.o = Linear(get(t["o"]), runtime)
+
+    def in_weights(self):
+        return list(self._in)
+
+    def in_width(self) -> int:
+        return 2 * (self.n_qk + self.n_v + self.H)
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in self._in) + self.o.nbytes()
+
+    def mix(self, proj: torch.Tensor, col: int, step, memory: MixerMemory) -> torch.Tensor:
+        """From the float32 projection rows `proj`, whose columns from `col` on are [q | k | v | g | i | f]: the normed, gated
+        heads [n, heads·vdim] in the engine's type, the input of `self.o`."""
+        act = self.runtime.empty(proj.shape[0], self.n_v)
+        k_col = col + self.n_qk
+        v_col = k_col + self.n_qk
+        g_col = v_col + self.n_v
+        i_col = g_col + self.n_v
+        kernels.matrix_memory(proj, col, k_col, v_col, g_col, i_col, i_col + self.H, self.i_bias, self.f_bias, self.cap, self.gain,
+                              self.eps, memory.state, step, self.H, self.dim, self.vdim, act)
+        return act
+
+    accumulates = True        # forward(..., residual=x) may add the branch into the float32 stream and return None
+
+    def forward(self, h: torch.Tensor, step, memory: MixerMemory, residual: Optional[torch.Tensor] = None):
+        if self.in_proj is None:
+            self.in_proj = fused_rows(self._in, self.runtime)
+        return project_out(self.o, self.mix(self.in_proj(h, torch.float32), 0, step, memory), residual)
+
+
 @register_part("mixer", "gated_linear_recurrence")
 class GatedLinearRecurrence(Part):
     """The recurrent block of Griffin (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for
@@ -407,12 +577,19 @@ class ParallelMixer(Part):
     def weight_bytes(self) -> int:
         return self.left.weight_bytes() + self.right.weight_bytes()
 
-    def forward(self, h: torch.Tensor, step, memory: MixerMemory) -> torch.Tensor:
+    accumulates = True        # forward(..., residual=x) may add the branch into the float32 stream and return None
+
+    def forward(self, h: torch.Tensor, step, memory: MixerMemory, residual: Optional[torch.Tensor] = None):
         n = h.shape[0]
         proj = self.in_proj(h, torch.float32)
         a_left = self.left.mix(proj, 0, step, memory)
         a_right = self.right.mix(proj, self.right_col, step, memory)
         lo, ro = self.left.o, self.right.o
+        if (residual is not None and a_left.dtype == a_right.dtype == torch.bfloat16 and lo.can_add_into_stream(n)
+                and ro.can_add_into_stream(n)):
+            lo.add_into(a_left, residual)
+            ro.add_into(a_right, residual)
+            return None
         if ro.can_add_into_stream(n) and a_right.dtype == torch.bfloat16:
             out = lo(a_left, torch.float32)
             ro.add_into(a_right, out)

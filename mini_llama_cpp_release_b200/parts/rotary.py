@@ -108,8 +108,10 @@ def stretched_frequencies(dims: int, base: float, scaling: Optional[dict]) -> Tu
 
     so that fast pairs keep their frequency and slow ones are divided by `factor`; cos and sin are both multiplied by
     0.1 · ln(factor) + 1.  With scaling = {factor} alone the stretching is linear: every frequency is divided by the
-    factor (positions count `factor` times slower) and the multiplier is one.  Returns (float32 frequencies [dims/2], that
-    multiplier).  Computed in float64, rounded once."""
+    factor (positions count `factor` times slower) and the multiplier is one.  With scaling = {factor, low, high, original}
+    (the form Llama 3.1 uses) a pair's wavelength l = 2π / f decides: below original/high its frequency stays, above
+    original/low it is divided by the factor, in between it is (1 - s) f / factor + s f with s = (original/l - low) / (high -
+    low); the multiplier is one.  Returns (float32 frequencies [dims/2], that multiplier).  Computed in float64, rounded once."""
     i = np.arange(dims // 2, dtype=np.float64)
     f = np.power(float(base), -2.0 * i / dims)
     if not scaling:
@@ -120,6 +122,14 @@ def stretched_frequencies(dims: int, base: float, scaling: Optional[dict]) -> Tu
         if factor <= 0:
             raise ValueError("rope scaling: factor must be positive")
         return (f / factor).astype(np.float32), 1.0
+    if "low" in scaling or "high" in scaling:
+        factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
+        if factor <= 0 or original <= 0 or low <= 0 or high < low:
+            raise ValueError("rope scaling: factor, original and low must be positive, and high not below low")
+        wave = 2.0 * math.pi / f
+        s = (original / wave - low) / (high - low) if high > low else np.zeros_like(f)
+        mixed = (1.0 - s) * f / factor + s * f
+        return np.where(wave < original / high, f, np.where(wave > original / low, f / factor, mixed)).astype(np.float32), 1.0
     factor, original = float(scaling["factor"]), float(scaling["original"])
     if factor <= 0 or original <= 0 or float(scaling["fast"]) <= 0 or float(scaling["slow"]) <= 0:
         raise ValueError("rope scaling: factor, original, fast and slow must be positive")

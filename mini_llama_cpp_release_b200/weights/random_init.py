@@ -32,6 +32,8 @@ def random_tensor(spec: TensorSpec, seed: int, dtype: torch.dtype, std: float = 
     g = torch.Generator(device="cpu")
     g.manual_seed(tensor_seed(seed, spec.name))
     shape = spec.default_shape if (spec.default_shape is not None and -1 in tuple(spec.shape)) else spec.shape
+    if spec.init == "distinct_rows":                  # a table of integers whose rows hold different numbers below `below`
+        return torch.rand(shape[0], spec.below, generator=g).argsort(dim=1)[:, :shape[1]].to(torch.int32).contiguous()
     if spec.init == "unit_interval":                  # a bound or a rate that lies between 0 and 1
         return (torch.rand(tuple(shape), generator=g, dtype=torch.float32) * 0.9 + 0.05).to(dtype)
     t = torch.randn(tuple(shape), generator=g, dtype=torch.float32) * std
@@ -54,7 +56,7 @@ def write_random_model(config: ModelConfig, folder: str, seed: int, dtype: torch
     spec = build_model_spec(cfg)
     parts = build_parts(spec).all_parts()
     wanted = [s for s in expected_tensors(parts).values() if s.stored and not s.optional]
-    layout = [(s.name, dtype, tuple(s.default_shape if (s.default_shape is not None and -1 in tuple(s.shape)) else s.shape))
+    layout = [(s.name, torch.int32 if s.role == "int_table" else dtype, tuple(s.default_shape if (s.default_shape is not None and -1 in tuple(s.shape)) else s.shape))
               for s in wanted]
     by_name: Dict[str, TensorSpec] = {s.name: s for s in wanted}
     save_safetensors_streamed(os.path.join(folder, "model.safetensors"), layout,
