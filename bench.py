@@ -7,6 +7,7 @@
     python bench.py --compare lonulix-w896 [--layers 6]   # the Lonulix design beside Kebesun layers of the same mixers and sizes
     python bench.py --compare nobonex-w896 [--layers 6]   # the Nobonex design beside the Kebesun preset of the same sizes
     python bench.py --compare bizenex-w896 [--layers 6]   # the Bizenex design beside Kebesun layers of the same mixers and sizes
+    python bench.py --compare betepel-w896 [--layers 6]   # the Betepel design beside Kebesun layers of the nearest mixers and the same sizes
 
 A "step" is one decode step of the whole batch.  The default run (`--config qwen2-0.5b`) has the layer sizes of a
 Qwen2-0.5B (24 layers, width 896, 14 query heads on 2 kv heads of size 64, feed-forward 4864, vocabulary 151936,
@@ -54,7 +55,9 @@ COMPARE = {"mepolix-w896": "qwen2-0.5b", "mepolix-w1536": "qwen2-1.5b", "mepolix
            # a Nobonex preset → the Kebesun preset of the same width, attention shape, feed-forward and experts (its closest design)
            "nobonex-w896": "kebesun-w896", "nobonex-w1536": "kebesun-w1536", "nobonex-w3584": "kebesun-w3584",
            # a Bizenex preset → the Kebesun layers of the same mixers, sizes and order (its closest design)
-           "bizenex-w896": "kebesun-al-w896", "bizenex-w1536": "kebesun-al-w1536", "bizenex-w3584": "kebesun-al-w3584"}
+           "bizenex-w896": "kebesun-al-w896", "bizenex-w1536": "kebesun-al-w1536", "bizenex-w3584": "kebesun-al-w3584",
+           # a Betepel preset → the Kebesun layers of the nearest mixers and the same sizes and order (its closest design)
+           "betepel-w896": "kebesun-ag-w896", "betepel-w1536": "kebesun-ag-w1536", "betepel-w3584": "kebesun-ag-w3584"}
 REF_DIR = os.path.join(ROOT, "baseline", "_ref")
 REF_SOURCE = os.environ.get("MLC_REFERENCE_SOURCE", "/root/reference")     # where the reference's checkout lies, if baseline/_ref is empty
 REF_PREFILL_TOKENS = 32
@@ -200,7 +203,7 @@ def main() -> int:
                     help="run one part only and print a short line (for profiling a small case)")
     ap.add_argument("--prompt-len", type=int, default=None, help="prompt length of the --only runs")
     ap.add_argument("--compare", default=None, choices=sorted(COMPARE),
-                    help="instead of the benchmark line: prompt and decode throughput of a Mepolix, Kebesun, Lonulix, Nobonex or Bizenex preset beside the "
+                    help="instead of the benchmark line: prompt and decode throughput of a Mepolix, Kebesun, Lonulix, Nobonex, Bizenex or Betepel preset beside the "
                          "preset of its closest design at the same width, head shape and feed-forward, at --layers layers each "
                          "(default 6)")
     args = ap.parse_args()

@@ -142,8 +142,12 @@ gla_walk_kernel(GlaArgs a) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             const int idx = tid + u * GLA_THREADS;
-            qs[idx] = (SILU ? silu_f(rq[u]) : rq[u]) * a.q_scale;
-            ks[idx] = SILU ? silu_f(rk[u]) : rk[u];
+            if (SILU && idx / DP < n_here) {          // (silu(0) = 0: nothing to do where there is no token)
+                rq[u] = silu_f(rq[u]);
+                rk[u] = silu_f(rk[u]);
+            }
+            qs[idx] = rq[u] * a.q_scale;
+            ks[idx] = rk[u];
             as[idx] = ra[u];
         }
 #pragma unroll

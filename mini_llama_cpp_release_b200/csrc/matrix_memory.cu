@@ -19,6 +19,25 @@
 
 namespace mlc {
 
+// ------------------------------------------------------------------ constant decay: what precedes the walk of a prompt
+// SiLU on columns [0, width) of every row, in place.  (A step of few tokens leaves it to the walk, whose blocks then each do
+// their own rows' and columns'; in a prompt every q and k would pass SiLU once per slab of columns.)
+template <int VEC>
+__global__ void silu_columns_kernel(float* __restrict__ rows, long long stride, int width, long long total) {
+    const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (idx >= total) return;
+    const long long t = idx / width;
+    float* p = rows + t * stride + (idx - t * width);
+    if constexpr (VEC == 4) {
+        float4 v = *reinterpret_cast<const float4*>(p);
+        v.x = v.x / (1.0f + expf(-v.x)); v.y = v.y / (1.0f + expf(-v.y));
+        v.z = v.z / (1.0f + expf(-v.z)); v.w = v.w / (1.0f + expf(-v.w));
+        *reinterpret_cast<float4*>(p) = v;
+    } else {
+        p[0] = p[0] / (1.0f + expf(-p[0]));
+    }
+}
+
 // ------------------------------------------------------------------ constant decay: what follows the walk
 // out[t] = (sum of the walk's slices) / rms(row) · gain · sigmoid(gate) · out_scale.  A block per token, a thread PIECES
 // pieces of VEC entries, the row in registers from its loads to its stores.
@@ -76,10 +95,10 @@ row_norm_gate_kernel(const float* __restrict__ o, int slices, long long slice_st
 }
 
 // ------------------------------------------------------------------ exponential gates: decays and input factors
-__device__ __forceinline__ void log_gates(const float* row, int i_col, int f_col, int h, const float* i_bias, const float* f_bias,
-                                          float cap, float inv_cap, float& li, float& lf) {
-    li = cap * tanhf((row[i_col + h] + i_bias[h]) * inv_cap);
-    const float x = cap * tanhf((row[f_col + h] + f_bias[h]) * inv_cap);
+// zi, zf: the gates' logits with their biases
+__device__ __forceinline__ void log_gates(float zi, float zf, float cap, float inv_cap, float& li, float& lf) {
+    li = cap * tanhf(zi * inv_cap);
+    const float x = cap * tanhf(zf * inv_cap);
     lf = fminf(x, 0.0f) - log1pf(expf(-fabsf(x)));
 }
 
@@ -109,7 +128,8 @@ __global__ void exp_gates_step_kernel(ExpGateArgs a) {
     float m = *ms;
     for (int t = a.cu_seqlens[seq]; t < a.cu_seqlens[seq + 1]; ++t) {
         float li, lf;
-        log_gates(a.proj + (long long)t * a.stride, a.i_col, a.f_col, h, a.i_bias, a.f_bias, a.cap, a.inv_cap, li, lf);
+        const float* row = a.proj + (long long)t * a.stride;
+        log_gates(row[a.i_col + h] + a.i_bias[h], row[a.f_col + h] + a.f_bias[h], a.cap, a.inv_cap, li, lf);
         const float next = fmaxf(lf + m, li);
         const long long at = (long long)t * a.H + h;
         a.decay[at] = expf(lf + m - next);
@@ -120,9 +140,9 @@ __global__ void exp_gates_step_kernel(ExpGateArgs a) {
     *ms = m;
 }
 
-// Longer runs: a block per (head, sequence) takes rounds of 256 x EG_RUN tokens, a thread EG_RUN tokens side by side.
-constexpr int EG_THREADS = 256;
-constexpr int EG_RUN = 8;
+// Longer runs: a block per (head, sequence) takes rounds of EG_THREADS x EG_RUN tokens, a thread EG_RUN tokens side by side.
+constexpr int EG_THREADS = 512;
+constexpr int EG_RUN = 4;
 
 __global__ void __launch_bounds__(EG_THREADS)
 exp_gates_scan_kernel(ExpGateArgs a) {
@@ -133,16 +153,25 @@ exp_gates_scan_kernel(ExpGateArgs a) {
     const int t0 = a.cu_seqlens[seq], t1 = a.cu_seqlens[seq + 1];
     float* ms = a.m_state + (long long)a.slots[seq] * a.state_stride + h;
     float m0 = *ms;
+    const float bi = a.i_bias[h], bf = a.f_bias[h];
     for (int c0 = t0; c0 < t1; c0 += EG_THREADS * EG_RUN) {
         const int first = c0 + threadIdx.x * EG_RUN;
         float li[EG_RUN], lf[EG_RUN];
         float A = 0.0f, B = -INFINITY;                    // the thread's run: m -> max(A + m, B)
+        float zi[EG_RUN], zf[EG_RUN];                     // all loads first (the last token's again where there is none)
 #pragma unroll
         for (int u = 0; u < EG_RUN; ++u) {
-            li[u] = -INFINITY;
-            lf[u] = 0.0f;                                 // no token: m stays as it is
-            if (first + u < t1)
-                log_gates(a.proj + (long long)(first + u) * a.stride, a.i_col, a.f_col, h, a.i_bias, a.f_bias, a.cap, a.inv_cap, li[u], lf[u]);
+            const float* row = a.proj + (long long)min(first + u, t1 - 1) * a.stride;
+            zi[u] = row[a.i_col + h];
+            zf[u] = row[a.f_col + h];
+        }
+#pragma unroll
+        for (int u = 0; u < EG_RUN; ++u) {
+            log_gates(zi[u] + bi, zf[u] + bf, a.cap, a.inv_cap, li[u], lf[u]);
+            if (first + u >= t1) {
+                li[u] = -INFINITY;
+                lf[u] = 0.0f;                             // no token: m stays as it is
+            }
         }
 #pragma unroll
         for (int u = 0; u < EG_RUN; ++u) {
@@ -269,11 +298,12 @@ static int launch_row_norm_gate(const float* o, int slices, long long slice_stri
 
 using namespace mlc;
 
-// Linear attention with a constant decay per head.  proj: float32 rows holding the logits of q, k (H x dim each), v and the
-// gate (H x vdim each) at their columns.  decay float32 [H], gain float32 [H*vdim].  state: float32, a slot's row holds
+// Linear attention with a constant decay per head.  proj: float32 rows holding the logits of q, k (H x dim each) and v
+// (H x vdim) side by side from column q_col on, and of the gate (H x vdim) at g_col; `silu_first` overwrites q, k and v with
+// their SiLU (one more launch) instead of leaving it to the walk.  decay float32 [H], gain float32 [H*vdim].  state: float32, a slot's row holds
 // H*vdim*dim floats ([head][column][row]).  rows: what mlc_gla_rows gave.  walk: float32 [ceil(dim / (8 * rows))][n][H*vdim]
 // scratch.  out [n][H*vdim] of out_dtype.
-extern "C" int mlc_decay_attention(const float* proj, long long proj_stride, int q_col, int k_col, int v_col, int g_col,
+extern "C" int mlc_decay_attention(float* proj, long long proj_stride, int q_col, int g_col, int silu_first,
                                    const float* decay, const float* gain, float eps, float out_scale, float* state,
                                    long long state_stride, const int* slots, const int* cu_seqlens, int n_seqs, int n_tokens,
                                    int H, int dim, int vdim, int rows, float* walk, void* out, int out_dtype, void* stream) {
@@ -281,13 +311,21 @@ extern "C" int mlc_decay_attention(const float* proj, long long proj_stride, int
     if (H <= 0 || vdim <= 0 || (long long)H * vdim > 16384 || rows < 1) return MLC_ERR_BAD_SIZE;
     if (out_dtype != MLC_DTYPE_F32 && out_dtype != MLC_DTYPE_BF16) return MLC_ERR_BAD_DTYPE;
     cudaStream_t s = (cudaStream_t)stream;
+    if (silu_first) {
+        const int width = H * (2 * dim + vdim);
+        const bool vec = (width & 3) == 0 && (proj_stride & 3) == 0 && (((uintptr_t)(proj + q_col)) & 15) == 0;
+        const long long total = (long long)n_tokens * width, items = vec ? total / 4 : total;
+        if (vec) silu_columns_kernel<4><<<(unsigned)((items + 255) / 256), 256, 0, s>>>(proj + q_col, proj_stride, width, total);
+        else silu_columns_kernel<1><<<(unsigned)((items + 255) / 256), 256, 0, s>>>(proj + q_col, proj_stride, width, total);
+        MLC_LAUNCH_CHECK();
+    }
     GlaArgs a = {};
     a.qk = a.vsrc = proj; a.qk_stride = a.v_stride = proj_stride;
-    a.q_col = q_col; a.k_col = k_col; a.v_col = v_col;
+    a.q_col = q_col; a.k_col = q_col + H * dim; a.v_col = q_col + 2 * H * dim;
     a.const_decay = decay; a.q_scale = 1.0f;
     a.state = state; a.state_stride = state_stride; a.slots = slots; a.cu_seqlens = cu_seqlens; a.out = walk;
     a.H = H; a.dim = dim; a.vdim = a.v_cols = vdim; a.qk_share = 1;
-    const int rc = gla_walk(a, n_seqs, n_tokens, rows, true, s);
+    const int rc = gla_walk(a, n_seqs, n_tokens, rows, !silu_first, s);
     if (rc != 0) return rc;
     const int slices = (dim + 8 * rows - 1) / (8 * rows), inner = H * vdim;
     const long long slice = (long long)n_tokens * inner;

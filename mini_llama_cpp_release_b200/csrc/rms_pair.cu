@@ -166,6 +166,7 @@ static cudaError_t launch_rms_pair(const PairNorm& a, const NormBranch& br, T* o
 }
 
 // ------------------------------------------------------------------ embedding behind a norm
+// A block per row, which it reads twice (the second time out of L1).
 template <typename T>
 __global__ void __launch_bounds__(1024)
 embed_rms_kernel(const T* __restrict__ table, const int* __restrict__ ids, int d, float scale, const float* __restrict__ gain, float eps,
@@ -182,6 +183,38 @@ embed_rms_kernel(const T* __restrict__ table, const int* __restrict__ ids, int d
     }
     const float f = 1.0f / sqrtf(block_sum(ss, scratch) / (float)d + eps);
     for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = to_float(row[i]) * scale * f * gain[i];
+}
+
+// Many rows: a warp per row, the row in registers (NV pieces of four entries per lane, d <= 128 * NV, d a multiple of 4).
+template <int NV>
+__global__ void __launch_bounds__(256)
+embed_rms_warp_kernel(const bf16* __restrict__ table, const int* __restrict__ ids, int n, int d, float scale,
+                      const float* __restrict__ gain, float eps, float* __restrict__ out) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int lane = threadIdx.x & 31;
+    const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (row >= n) return;
+    const uint2* src = reinterpret_cast<const uint2*>(table + (long long)ids[row] * d);
+    const int d4 = d >> 2;
+    float v[NV][4];
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = lane + 32 * k;
+        const uint2 q = i < d4 ? src[i] : make_uint2(0u, 0u);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+        v[k][0] = a.x * scale; v[k][1] = a.y * scale; v[k][2] = b.x * scale; v[k][3] = b.y * scale;
+        ss += (v[k][0] * v[k][0] + v[k][1] * v[k][1]) + (v[k][2] * v[k][2] + v[k][3] * v[k][3]);
+    }
+    const float f = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = lane + 32 * k;
+        if (i >= d4) continue;
+        store_scaled<float, 4>(out + (long long)row * d + 4 * i, v[k], f, gain + 4 * i);
+    }
 }
 
 // ------------------------------------------------------------------ differential attention: what follows the two maps
@@ -284,7 +317,12 @@ extern "C" int mlc_embed_rms(const void* table, int table_dtype, const int* ids,
     if (n <= 0) return 0;
     if (d <= 0) return MLC_ERR_BAD_SIZE;
     cudaError_t e;
-    if (table_dtype == MLC_DTYPE_F32)
+    const int nv = ((d >> 2) + 31) / 32;
+    if (table_dtype == MLC_DTYPE_BF16 && n >= 256 && (d & 3) == 0 && nv <= 32 &&
+        ((((uintptr_t)table) | ((uintptr_t)gain) | ((uintptr_t)out)) & 15) == 0) {
+        auto k = nv <= 4 ? embed_rms_warp_kernel<4> : nv <= 8 ? embed_rms_warp_kernel<8> : nv <= 16 ? embed_rms_warp_kernel<16> : embed_rms_warp_kernel<32>;
+        e = launch_pdl(k, dim3((n + 7) / 8), dim3(256), 0, (cudaStream_t)stream, (const bf16*)table, ids, n, d, scale, gain, eps, out);
+    } else if (table_dtype == MLC_DTYPE_F32)
         e = launch_pdl(embed_rms_kernel<float>, dim3(n), dim3(row_block(d)), 0, (cudaStream_t)stream, (const float*)table, ids, d, scale, gain, eps, out);
     else if (table_dtype == MLC_DTYPE_BF16)
         e = launch_pdl(embed_rms_kernel<bf16>, dim3(n), dim3(row_block(d)), 0, (cudaStream_t)stream, (const bf16*)table, ids, d, scale, gain, eps, out);

@@ -112,7 +112,7 @@ def core() -> ctypes.CDLL:
             "mlc_moe_route": [P, I, P, P, I, I, I, I, I, P, P, P],
             "mlc_moe_plan": [P, I, I, I, I, I, P, P, P, P],
             "mlc_moe_plan_table": [P, P, F, P, I, I, I, I, I, P, P, P, P],
-            "mlc_decay_attention": [P, LL, I, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, I, I, P, P, I, P],
+            "mlc_decay_attention": [P, LL, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, I, I, P, P, I, P],
             "mlc_matrix_memory": [P, LL, I, I, I, I, I, I, P, P, F, P, F, P, LL, P, P, I, I, I, I, I, I, I, P, P, P, I, P],
             "mlc_rms_pair": [P, P, I, P, P, P, I, P, P, F, I, I, P, P, I, P],
             "mlc_embed_rms": [P, I, P, I, I, F, P, F, P, P],
@@ -873,12 +873,12 @@ def state_space(proj: torch.Tensor, z_col: int, dt_col: int, xbc: torch.Tensor, 
 
 
 # ------------------------------------------------------------------ memories that decay per head (csrc/matrix_memory.cu)
-def decay_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_col: int, decay: torch.Tensor, gain: torch.Tensor,
+def decay_attention(proj: torch.Tensor, q_col: int, g_col: int, decay: torch.Tensor, gain: torch.Tensor,
                     eps: float, out_scale: float, state: torch.Tensor, step, heads: int, dim: int, vdim: int, out: torch.Tensor) -> None:
     """Linear attention with one constant decay per head over the step's tokens: S <- decay S + silu(k) silu(v)T,
     o = ST silu(q); then all heads together divided by their root mean square, times `gain`, times sigmoid(gate), times
-    `out_scale`.  q, k (heads x dim), v and the gate (heads x vdim) in the float32 rows `proj`; decay float32 [heads]; gain float32
-    [heads*vdim]; state float32 [slots, heads*vdim*dim]; out [n, heads*vdim] in the engine's type."""
+    `out_scale`.  The logits of q, k (heads x dim each) and v (heads x vdim) side by side in the float32 rows `proj` from q_col
+    on (overwritten in a step of many tokens), the gate's (heads x vdim) at g_col; decay float32 [heads]; gain float32 [heads*vdim]; state float32 [slots, heads*vdim*dim]; out [n, heads*vdim] in the engine's type."""
     require_cuda(decay, gain, out)
     _require_rows(state)
     _require_rows(proj)
@@ -889,11 +889,12 @@ def decay_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_co
     assert decay.dtype == gain.dtype == torch.float32 and decay.numel() == heads and gain.numel() == heads * vdim
     assert state.shape[1] == heads * vdim * dim and tuple(out.shape) == (n, heads * vdim)
     walk = torch.empty(slices * n * heads * vdim, dtype=torch.float32, device=out.device)
-    _check(lib.mlc_decay_attention(proj.data_ptr(), proj.stride(0), q_col, k_col, v_col, g_col, decay.data_ptr(), gain.data_ptr(),
+    silu_first = n > 64                 # a prompt: SiLU once per value, not once per block of the walk that reads it
+    _check(lib.mlc_decay_attention(proj.data_ptr(), proj.stride(0), q_col, g_col, 1 if silu_first else 0, decay.data_ptr(), gain.data_ptr(),
                                    float(eps), float(out_scale), state.data_ptr(), state.stride(0), step.slots.data_ptr(),
                                    step.cu_seqlens.data_ptr(), step.n_seqs, n, heads, dim, vdim, rows, walk.data_ptr(),
                                    out.data_ptr(), dtype_code(out.dtype), _stream()), "linear attention with a constant decay")
-    count_launches(1)
+    count_launches(2 if silu_first else 1)
 
 
 def matrix_memory(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_col: int, i_col: int, f_col: int, i_bias: torch.Tensor,

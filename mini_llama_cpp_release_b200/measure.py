@@ -142,6 +142,41 @@ def _bizenex(width: int, ff: int, heads: int, kv_heads: int, head: int, n_layers
     return dict(top, layers=layers)
 
 
+def _betepel(width: int, ff: int, heads: int, kv_heads: int, head: int, n_layers: int, vocab: int, design: str = "Betepel") -> Dict[str, Any]:
+    """Betepel layers of real width in a cycle of six: differential attention, windowed attention beside constant-decay linear
+    attention, a matrix memory, differential attention, the same on the keys and values of the layer before it, a matrix memory;
+    every layer has experts.  The width and the attention's head count and head size are the Qwen2 preset's of the same width (a
+    differential head has two maps of half its size); windows of 1,024 keys with the first four kept, the linear layers' shape
+    (half the heads, values twice as wide) and the experts (eight of half its dense feed-forward) are the Kebesun preset's; a
+    token passes one routed expert and a shared one of the same size where that preset routes it to two.
+    `design="Kebesun"` gives that design's layers of the nearest mixers and the same sizes in the same order (windowed attention,
+    windowed attention, gated linear attention, windowed attention twice, gated linear attention): the model the Betepel preset
+    is timed beside."""
+    mask = {"size": 1024, "keep_first": 4}
+    lin = {"heads": max(1, heads // 2), "dim": head, "vdim": 2 * head}
+    experts = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+    if design == "Kebesun":
+        att = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5,
+               "rot": {"dims": head, "base": 1000000.0, "scaling": {"factor": 4.0}}, "mask": mask}
+        gla = dict(lin, tau=16.0)
+        cycle = [("attention", att), ("attention", att), ("gla", gla), ("attention", att), ("attention", att), ("gla", gla)]
+        return {"architecture": "Kebesun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                "layers": [{"type": t, "mixer": dict(m), "mlp": dict(experts)} for t, m in (cycle[i % 6] for i in range(n_layers))]}
+    diff = {"heads": heads, "kv_heads": kv_heads, "dim": head // 2, "vdim": head, "scale": (head // 2) ** -0.5, "diff": 0.55, "mask": mask,
+            "rot": {"dims": head // 2, "base": 1000000.0, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5, "mask": {"size": 1024},
+                    "rot": {"dims": head, "base": 10000.0}},
+           "right": dict(lin, decay=[round(1.0 - 2.0 ** -(3 + 5 * h / lin["heads"]), 6) for h in range(lin["heads"])]),
+           "left_scale": 0.9, "right_scale": 1.2}
+    experts = dict(experts, router={"experts": 8, "top": 1}, shared={"ff": ff // 2})
+    layers = []
+    for i in range(n_layers):
+        t, m = [("attention", diff), ("parallel", par), ("mlstm", dict(lin, gate_cap=12.0)), ("attention", diff),
+                ("attention", dict(diff, kv_from=i - 1)), ("mlstm", dict(lin, gate_cap=12.0))][i % 6]
+        layers.append({"type": t, "mixer": dict(m), "mlp": dict(experts)})
+    return {"architecture": "Betepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": layers}
+
+
 PRESETS: Dict[str, Dict[str, Any]] = {
     "tiny-a": dict(_QWEN2, hidden_size=64, intermediate_size=176, num_hidden_layers=2, num_attention_heads=4,
                    num_key_value_heads=2, head_dim=16, vocab_size=512, max_position_embeddings=256, rope_theta=10000.0,
@@ -184,6 +219,13 @@ PRESETS: Dict[str, Dict[str, Any]] = {
     "kebesun-al-w896": _bizenex(896, 4864, 14, 2, 64, 24, 151936, design="Kebesun"),
     "kebesun-al-w1536": _bizenex(1536, 8960, 12, 2, 128, 24, 151936, design="Kebesun"),
     "kebesun-al-w3584": _bizenex(3584, 18944, 28, 4, 128, 24, 152064, design="Kebesun"),
+    # the Betepel design at the same widths, and the Kebesun layers of the nearest mixers it is timed beside (see `_betepel`)
+    "betepel-w896": _betepel(896, 4864, 14, 2, 64, 24, 151936),
+    "betepel-w1536": _betepel(1536, 8960, 12, 2, 128, 24, 151936),
+    "betepel-w3584": _betepel(3584, 18944, 28, 4, 128, 24, 152064),
+    "kebesun-ag-w896": _betepel(896, 4864, 14, 2, 64, 24, 151936, design="Kebesun"),
+    "kebesun-ag-w1536": _betepel(1536, 8960, 12, 2, 128, 24, 151936, design="Kebesun"),
+    "kebesun-ag-w3584": _betepel(3584, 18944, 28, 4, 128, 24, 152064, design="Kebesun"),
 }
 
 FALLBACK_PEAKS = dict(hbm_gbs=6650.0, bf16_tflops=1590.0)

@@ -346,9 +346,7 @@ class DecayAttention(Part):
         """From the float32 projection rows `proj`, whose columns from `col` on are [q | k | v | g]: the normed, gated heads
         [n, heads·vdim] in the engine's type, the input of `self.o`."""
         act = self.runtime.empty(proj.shape[0], self.n_v)
-        k_col = col + self.n_qk
-        v_col = k_col + self.n_qk
-        kernels.decay_attention(proj, col, k_col, v_col, v_col + self.n_v, self.decay, self.gain, self.eps, self.out_scale,
+        kernels.decay_attention(proj, col, col + 2 * self.n_qk + self.n_v, self.decay, self.gain, self.eps, self.out_scale,
                                 memory.state, step, self.H, self.dim, self.vdim, act)
         return act
 

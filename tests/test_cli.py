@@ -108,7 +108,8 @@ def test_model_comes_from_a_folder_a_file_or_a_random_configuration(tmp_path, mo
     folder_b, _ = cli.resolve_model(parse("--random", str(tmp_path / "mine" / "config.json")))
     assert helpers.ml.ModelConfig.from_folder(folder_b).vocab_size == 1000
     # the presets are the configurations the measurements are quoted on
-    assert sorted(measure.PRESETS) == ["bizenex-w1536", "bizenex-w3584", "bizenex-w896", "kebesun-al-w1536", "kebesun-al-w3584",
+    assert sorted(measure.PRESETS) == ["betepel-w1536", "betepel-w3584", "betepel-w896", "bizenex-w1536", "bizenex-w3584", "bizenex-w896",
+                                       "kebesun-ag-w1536", "kebesun-ag-w3584", "kebesun-ag-w896", "kebesun-al-w1536", "kebesun-al-w3584",
                                        "kebesun-al-w896", "kebesun-lg-w1536", "kebesun-lg-w3584", "kebesun-lg-w896", "kebesun-w1536", "kebesun-w3584",
                                        "kebesun-w896", "lonulix-w1536", "lonulix-w3584", "lonulix-w896", "mepolix-w1536",
                                        "mepolix-w3584", "mepolix-w896", "nobonex-w1536", "nobonex-w3584", "nobonex-w896", "qwen2-0.5b",
