@@ -503,7 +503,8 @@ def model_prefill_flops(model, lengths: Sequence[int]) -> float:
             if isinstance(part, GQAttention):
                 # a window bounds the keys a row reads
                 w = getattr(part, "window", None)
-                total += part.H * 2.0 * part.hd * (squares if not w else sum(float(n) * min(n, 2 * w) for n in lengths))
+                entries = getattr(part, "useful_entries", 2 * part.hd)         # of a query row and a value row together
+                total += part.H * float(entries) * (squares if not w else sum(float(n) * min(n, 2 * w) for n in lengths))
             if hasattr(part, "flops_per_token"):
                 total += T * part.flops_per_token()
     return total + 2.0 * model.config.vocab_size * model.parts.head.hidden * len(lengths)

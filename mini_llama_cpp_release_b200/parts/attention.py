@@ -431,6 +431,7 @@ class DifferentialAttention(SinkAttention):
         self.H = self.MAPS * self.heads                               # query heads as the attention kernels see them
         self.dim, self.vdim = int(head_dim), int(v_head_dim)
         self.hd = (max(self.MAPS * self.dim, self.vdim) + 15) // 16 * 16
+        self.useful_entries = self.dim + self.vdim                    # what a query row multiplies but zeros (for the work's count)
         if self.hd > 512:
             raise ValueError(f"differential attention: 2 · dim and vdim up to 512 are supported, got dim {head_dim} and vdim {v_head_dim}")
         if not scale > 0:
